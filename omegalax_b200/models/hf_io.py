@@ -21,6 +21,18 @@ def load_hf_config(file_dir: str | os.PathLike) -> dict[str, Any]:
     return json.loads(path.read_text())
 
 
+def safetensors_shapes(source: str | os.PathLike) -> dict[str, tuple[int, ...]]:
+    """Tensor name -> shape of the checkpoint in directory ``source``; empty when there is none."""
+    from safetensors import safe_open
+
+    p = Path(str(source)).expanduser()
+    out: dict[str, tuple[int, ...]] = {}
+    for f in sorted(p.glob("*.safetensors")) if p.is_dir() else []:
+        with safe_open(str(f), framework="pt") as sf:
+            out.update({k: tuple(sf.get_slice(k).get_shape()) for k in sf.keys()})
+    return out
+
+
 def load_hf_config_from_source(source: str | os.PathLike) -> dict[str, Any]:
     """``source`` is a model directory, a path to a config.json, or a hub repo id.  Hub ids
     are resolved through the local HuggingFace cache only (``huggingface_hub`` downloads

@@ -277,11 +277,15 @@ class Qwen3(nn.Module):
         return ForwardCtx(B=B, T=T, sin=sin, cos=cos, cu_seqlens=cu, segment_ids=segment_ids,
                           k_start=k_start, positions=positions)
 
+    def logits(self, hidden):
+        return self.lm_head(hidden)
+
     @torch.no_grad()
-    def decode_paged(self, token_ids, segment_ids, cache):
+    def decode_paged(self, token_ids, segment_ids, cache, select=None):
         """Prefill or one decode step against a ``PagedKVCache`` (CUDA bf16).  Only real tokens
         are processed and stored; returns the final hidden state of every sequence's last new
-        token, [B, D] (zeros for sequences without a new token)."""
+        token, [B, D] (zeros for sequences without a new token), or, with the bool mask ``select``
+        [B, T], of the marked tokens in order."""
         from ...ops import kernels as K
 
         cfg = self.cfg
@@ -331,6 +335,8 @@ class Qwen3(nn.Module):
             x = layer.mlp(hh, residual=x)[0] if layer.is_moe else layer.mlp(hh, residual=x)
         cache.advance(new_tokens)
         x = self.final_norm(x)
+        if select is not None:
+            return x[(select.to(dev) & real)[real]]
         out = torch.zeros(B, x.shape[1], dtype=x.dtype, device=dev)
         has = counts > 0
         out[has] = x[last[has]]

@@ -19,6 +19,11 @@
 // Sequences are packed: row r of sequence b is global row cu_seqlens[b] + r.  Q/O are
 // [rows, H, HD]; K/V are [rows, G, HD] with arbitrary row pitch (they may be slices of a
 // fused QKV buffer).  LSE is written as [H, rows] in natural-log units for the backward.
+//
+// Query / key width and value width are separate (QB and VB blocks of 64 channels), and a head's
+// channels may come from two tensors: blocks [0, nb1) of Q and K through the first pair of maps, the
+// rest through the second, whose key part is shared by all heads (latent attention: expanded keys
+// plus one rotated part).  Widths that are not multiples of 64 are zero-filled by the TMA boxes.
 #include "host_utils.h"
 #include "sm100_common.cuh"
 
@@ -35,26 +40,32 @@ struct AttnFwdArgs {
   int H, G;
   int causal;
   float scale_log2;       // softmax scale * log2(e)
+  int nb1;                // 64-channel blocks of Q / K read through the first pair of maps
+  int vdim;               // value channels that exist (<= 64 * VB)
   int* status;
 };
 
-template <int HD>
+template <int QB, int VB, int KST, int VST>
 struct AttnFwdSmem {
-  static constexpr int kTile = 128 * HD * 2;          // one 128-row operand tile
+  static constexpr int kQTile = 128 * QB * 64 * 2;    // one 128-row query / key tile
+  static constexpr int kVTile = 128 * VB * 64 * 2;
   static constexpr int kQOff = 0;                     // 2 tiles
-  static constexpr int kKOff = 2 * kTile;             // 2 stages
-  static constexpr int kVOff = 4 * kTile;             // 2 stages
-  static constexpr int kBarOff = 6 * kTile;
+  static constexpr int kKOff = 2 * kQTile;            // KST stages
+  static constexpr int kVOff = (2 + KST) * kQTile;    // VST stages
+  static constexpr int kBarOff = kVOff + VST * kVTile;
   static constexpr int kTotal = kBarOff + 256 + 1024;
 };
 
-template <int HD>
+template <int QB, int VB, int KST, int VST>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                const __grid_constant__ CUtensorMap tmV, const AttnFwdArgs p) {
+                const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQ2,
+                const __grid_constant__ CUtensorMap tmK2, const AttnFwdArgs p) {
+  static_assert(VB <= 2 && KST <= 2 && VST <= 2, "TMEM columns and barrier slots");
+  constexpr int VD = VB * 64;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-  using L = AttnFwdSmem<HD>;
+  using L = AttnFwdSmem<QB, VB, KST, VST>;
   uint64_t* q_full = (uint64_t*)(smem + L::kBarOff);  // [2]
   uint64_t* k_full = q_full + 2;                      // [2]
   uint64_t* v_full = k_full + 2;                      // [2]
@@ -110,7 +121,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
-  // TMEM columns: S0 [0,128) S1 [128,256) O0 [256,256+HD) O1 [384,384+HD)
+  // TMEM columns: S0 [0,128) S1 [128,256) O0 [256,256+VD) O1 [384,384+VD)
 
   if (warp < 4) {
     setmaxnreg_dec<40>();
@@ -122,48 +133,51 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
       for (int w = 0; w < 2; ++w) {
         if (n_w[w] > 0) {
-          mbar_expect_tx(&q_full[w], L::kTile);
+          mbar_expect_tx(&q_full[w], L::kQTile);
 #pragma unroll
-          for (int kb = 0; kb < HD / 64; ++kb)
-            tma_load_3d(smem + L::kQOff + w * L::kTile + kb * 16384, &tmQ, &q_full[w], kb * 64, h,
-                        seq_start + q0 + w * 128);
+          for (int kb = 0; kb < QB; ++kb) {
+            const bool first = kb < p.nb1;
+            tma_load_3d(smem + L::kQOff + w * L::kQTile + kb * 16384, first ? &tmQ : &tmQ2, &q_full[w],
+                        (first ? kb : kb - p.nb1) * 64, h, seq_start + q0 + w * 128);
+          }
         }
       }
       bool ok = true;
       for (int j = 0; j < n && ok; ++j) {
-        const int s = j & 1;
-        const uint32_t ph = ((j >> 1) & 1) ^ 1;
-        ok = mbar_wait(&k_empty[s], ph, abort_flag, p.status, OB_ERR_WAIT_EMPTY);
+        const int sk = j % KST, sv = j % VST;
+        ok = mbar_wait(&k_empty[sk], ((j / KST) & 1) ^ 1, abort_flag, p.status, OB_ERR_WAIT_EMPTY);
         if (!ok) break;
-        mbar_expect_tx(&k_full[s], L::kTile);
+        mbar_expect_tx(&k_full[sk], L::kQTile);
 #pragma unroll
-        for (int kb = 0; kb < HD / 64; ++kb)
-          tma_load_3d(smem + L::kKOff + s * L::kTile + kb * 16384, &tmK, &k_full[s], kb * 64, g,
-                      seq_start + j * 128);
-        ok = mbar_wait(&v_empty[s], ph, abort_flag, p.status, OB_ERR_WAIT_EMPTY);
+        for (int kb = 0; kb < QB; ++kb) {
+          const bool first = kb < p.nb1;
+          tma_load_3d(smem + L::kKOff + sk * L::kQTile + kb * 16384, first ? &tmK : &tmK2, &k_full[sk],
+                      (first ? kb : kb - p.nb1) * 64, first ? g : 0, seq_start + j * 128);
+        }
+        ok = mbar_wait(&v_empty[sv], ((j / VST) & 1) ^ 1, abort_flag, p.status, OB_ERR_WAIT_EMPTY);
         if (!ok) break;
-        mbar_expect_tx(&v_full[s], L::kTile);
+        mbar_expect_tx(&v_full[sv], L::kVTile);
 #pragma unroll
-        for (int kb = 0; kb < HD / 64; ++kb)
-          tma_load_3d(smem + L::kVOff + s * L::kTile + kb * 16384, &tmV, &v_full[s], kb * 64, g,
+        for (int kb = 0; kb < VB; ++kb)
+          tma_load_3d(smem + L::kVOff + sv * L::kVTile + kb * 16384, &tmV, &v_full[sv], kb * 64, g,
                       seq_start + j * 128);
       }
     } else if (warp == 1 && lane == 0) {
       // -------------------------------------------------------- MMA issuer
       constexpr uint32_t idesc_s = make_idesc_bf16(128, 128, 0, 0);
-      constexpr uint32_t idesc_o = make_idesc_bf16(128, HD, 0, 1);
+      constexpr uint32_t idesc_o = make_idesc_bf16(128, VD, 0, 1);
       auto issue_s = [&](int w, int s) {
-        const uint32_t qa = smem_u32(smem + L::kQOff + w * L::kTile);
-        const uint32_t ka = smem_u32(smem + L::kKOff + s * L::kTile);
-#pragma unroll
-        for (int k = 0; k < HD / 16; ++k) {
+        const uint32_t qa = smem_u32(smem + L::kQOff + w * L::kQTile);
+        const uint32_t ka = smem_u32(smem + L::kKOff + s * L::kQTile);
+#pragma unroll (QB > 2 ? 4 : QB * 4)
+        for (int k = 0; k < QB * 4; ++k) {
           const uint32_t off = (k >> 2) * 16384 + (k & 3) * 32;
           umma_ss(tmem_base + w * 128, make_smem_desc(qa + off, 16, 1024),
                   make_smem_desc(ka + off, 16, 1024), idesc_s, k > 0 ? 1u : 0u);
         }
       };
       auto issue_pv = [&](int w, int s, bool first) {
-        const uint32_t va = smem_u32(smem + L::kVOff + s * L::kTile);
+        const uint32_t va = smem_u32(smem + L::kVOff + s * L::kVTile);
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
           // 16 keys per step: A = 8 packed TMEM columns, B advances 16 rows of 128 bytes
@@ -183,8 +197,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       }
       if (ok) umma_commit(&k_empty[0]);
       for (int j = 0; j < n && ok; ++j) {
-        const int s = j & 1;
-        ok = mbar_wait(&v_full[s], (j >> 1) & 1, abort_flag, p.status, OB_ERR_WAIT_FULL);
+        const int s = j % VST, kn = (j + 1) % KST;     // stage of this V tile and of the next K tile
+        ok = mbar_wait(&v_full[s], (j / VST) & 1, abort_flag, p.status, OB_ERR_WAIT_FULL);
         if (!ok) break;
         bool k_next_ready = false;
         for (int w = 0; w < 2 && ok; ++w) {
@@ -196,19 +210,18 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           umma_commit(&o_full[w]);
           if (j + 1 < n_w[w]) {
             if (!k_next_ready) {
-              ok = mbar_wait(&k_full[(j + 1) & 1], ((j + 1) >> 1) & 1, abort_flag, p.status,
-                             OB_ERR_WAIT_FULL);
+              ok = mbar_wait(&k_full[kn], ((j + 1) / KST) & 1, abort_flag, p.status, OB_ERR_WAIT_FULL);
               if (!ok) break;
               tc_fence_after();
               k_next_ready = true;
             }
-            issue_s(w, (j + 1) & 1);
+            issue_s(w, kn);
             umma_commit(&s_full[w]);
           }
         }
         if (!ok) break;
         umma_commit(&v_empty[s]);
-        if (j + 1 < n) umma_commit(&k_empty[(j + 1) & 1]);
+        if (j + 1 < n) umma_commit(&k_empty[kn]);
       }
     }
   } else {
@@ -262,7 +275,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           if (!ok) break;
           tc_fence_after();
 #pragma unroll 1
-          for (int c = 0; c < HD / 32; ++c) {
+          for (int c = 0; c < VD / 32; ++c) {
             uint32_t v[32];
             tmem_ld32(o_addr + c * 32, v);
             tmem_ld_wait();
@@ -304,13 +317,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (lane == 0) mbar_arrive(&p_ready[w]);
     }
     // the accumulator of the last tile
-    float o_acc[HD];
+    float o_acc[VD];
     if (ok && nj > 0) {
       ok = mbar_wait(&o_full[w], (nj - 1) & 1, abort_flag, p.status, OB_ERR_WAIT_TMEM_FULL);
       if (ok) {
         tc_fence_after();
 #pragma unroll
-        for (int c = 0; c < HD / 32; ++c) {
+        for (int c = 0; c < VD / 32; ++c) {
           uint32_t v[32];
           tmem_ld32(o_addr + c * 32, v);
           tmem_ld_wait();
@@ -323,9 +336,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     if (ok && nj > 0 && qpos < seqlen) {
       const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
       const long long grow = (long long)seq_start + qpos;
-      bf16* op = p.out + grow * p.o_row_stride + (long long)h * HD;
+      bf16* op = p.out + grow * p.o_row_stride + (long long)h * p.vdim;
 #pragma unroll
-      for (int i = 0; i < HD / 8; ++i) {
+      for (int i = 0; i < VD / 8; ++i) {
+        if (i * 8 >= p.vdim) break;
         uint4 q;
         q.x = pack_bf16(o_acc[i * 8 + 0] * inv_l, o_acc[i * 8 + 1] * inv_l);
         q.y = pack_bf16(o_acc[i * 8 + 2] * inv_l, o_acc[i * 8 + 3] * inv_l);
@@ -352,8 +366,21 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   }
 }
 
+template <int QB, int VB, int KST, int VST>
+static int run_attn_fwd(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmQ2,
+                        const CUtensorMap& tmK2, const AttnFwdArgs& a, int B, int max_seqlen, cudaStream_t stream) {
+  using L = AttnFwdSmem<QB, VB, KST, VST>;
+  static_assert(L::kTotal <= 227 * 1024, "shared memory");
+  auto kern = attn_fwd_kernel<QB, VB, KST, VST>;
+  OB_ENSURE_DYN_SMEM(kern, L::kTotal);
+  dim3 grid((max_seqlen + 255) / 256, a.H, B);
+  kern<<<grid, kAttnThreads, L::kTotal, stream>>>(tmQ, tmK, tmV, tmQ2, tmK2, a);
+  OB_CHECK_LAUNCH();
+  return 0;
+}
+
 template <int HD>
-static int launch_attn_fwd(const void* q, const void* k, const void* v, const AttnFwdArgs& a,
+static int launch_attn_fwd(const void* q, const void* k, const void* v, AttnFwdArgs a,
                            long long q_row_stride, long long k_row_stride, long long v_row_stride,
                            int B, int max_seqlen, cudaStream_t stream) {
   CUtensorMap tmQ, tmK, tmV;
@@ -366,12 +393,9 @@ static int launch_attn_fwd(const void* q, const void* k, const void* v, const At
   e = make_tmap_3d(&tmV, v, HD, a.G, a.total_rows, (uint64_t)HD * 2, (uint64_t)v_row_stride * 2, 64,
                    1, 128);
   if (e) return 3500 + e;
-  auto kern = attn_fwd_kernel<HD>;
-  OB_ENSURE_DYN_SMEM(kern, AttnFwdSmem<HD>::kTotal);
-  dim3 grid((max_seqlen + 255) / 256, a.H, B);
-  kern<<<grid, kAttnThreads, AttnFwdSmem<HD>::kTotal, stream>>>(tmQ, tmK, tmV, a);
-  OB_CHECK_LAUNCH();
-  return 0;
+  a.nb1 = HD / 64;
+  a.vdim = HD;
+  return run_attn_fwd<HD / 64, HD / 64, 2, 2>(tmQ, tmK, tmV, tmQ, tmK, a, B, max_seqlen, stream);
 }
 
 // attention_fwd256_sm100.cu
@@ -415,6 +439,57 @@ int ob_attn_fwd(const void* q, const void* k, const void* v, void* out, float* l
   if (HD == 256)
     return launch_attn_fwd256(q, k, v, out, lse, cu_seqlens, B, max_seqlen, total_rows, H, G, q_row_stride,
                               k_row_stride, v_row_stride, o_row_stride, scale, causal, status, stream);
+  return 6005;
+}
+
+// Causal attention whose heads have a first part of d1 channels (own key per head) and a second part
+// of d2 channels (one key for all heads), and vdim value channels; forward only.
+//   q  [rows, H, d1 + d2] (pitch q_row_stride)       out [rows, H, vdim]
+//   k1 [rows, H, d1] (pitch k_row_stride)            v   [rows, H, vdim] (pitch v_row_stride)
+//   k2 [rows, d2] (pitch k2_row_stride)
+// Every width and pitch is a multiple of 8 elements.  Returns 6005 for widths without an instantiation
+// (ceil(d1/64) + ceil(d2/64) > 4, or vdim > 128).
+int ob_attn_fwd_two_part(const void* q, const void* k1, const void* k2, const void* v, void* out, const int* cu_seqlens,
+                         int B, int max_seqlen, long long total_rows, int H, int d1, int d2, int vdim,
+                         long long q_row_stride, long long k_row_stride, long long k2_row_stride, long long v_row_stride,
+                         float scale, int* status, cudaStream_t stream) {
+  if (B <= 0 || total_rows <= 0) return 0;
+  if ((q_row_stride & 7) || (k_row_stride & 7) || (k2_row_stride & 7) || (v_row_stride & 7) || (d1 & 7) || (d2 & 7) || (vdim & 7))
+    return 6001;
+  if ((((uintptr_t)q) | ((uintptr_t)k1) | ((uintptr_t)k2) | ((uintptr_t)v) | ((uintptr_t)out)) & 15) return 6002;
+  AttnFwdArgs a = {};
+  a.cu_seqlens = cu_seqlens;
+  a.out = (bf16*)out;
+  a.o_row_stride = (long long)H * vdim;
+  a.total_rows = total_rows;
+  a.H = H; a.G = H; a.causal = 1;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.nb1 = (d1 + 63) / 64;
+  a.vdim = vdim;
+  a.status = status;
+  const int qb = a.nb1 + (d2 + 63) / 64, vb = (vdim + 63) / 64;
+  if (qb > 4 || vb > 2) return 6005;
+  const uint64_t head_bytes = (uint64_t)(d1 + d2) * 2;
+  CUtensorMap tmQ, tmK, tmV, tmQ2, tmK2;
+  int e = make_tmap_3d(&tmQ, q, d1, H, total_rows, head_bytes, (uint64_t)q_row_stride * 2, 64, 1, 128);
+  if (!e) e = make_tmap_3d(&tmQ2, (const bf16*)q + d1, d2, H, total_rows, head_bytes, (uint64_t)q_row_stride * 2, 64, 1, 128);
+  if (e) return 2000 + e;
+  e = make_tmap_3d(&tmK, k1, d1, H, total_rows, (uint64_t)d1 * 2, (uint64_t)k_row_stride * 2, 64, 1, 128);
+  if (!e) e = make_tmap_3d(&tmK2, k2, d2, 1, total_rows, (uint64_t)k2_row_stride * 2, (uint64_t)k2_row_stride * 2, 64, 1, 128);
+  if (e) return 3000 + e;
+  e = make_tmap_3d(&tmV, v, vdim, H, total_rows, (uint64_t)vdim * 2, (uint64_t)v_row_stride * 2, 64, 1, 128);
+  if (e) return 3500 + e;
+#define OB_TP(Q, V, KS, VS) return run_attn_fwd<Q, V, KS, VS>(tmQ, tmK, tmV, tmQ2, tmK2, a, B, max_seqlen, stream)
+  if (vb == 1) {
+    if (qb == 2) OB_TP(2, 1, 2, 2);
+    if (qb == 3) OB_TP(3, 1, 2, 2);
+    if (qb == 4) OB_TP(4, 1, 1, 2);
+  } else {
+    if (qb == 2) OB_TP(2, 2, 2, 2);
+    if (qb == 3) OB_TP(3, 2, 2, 1);
+    if (qb == 4) OB_TP(4, 2, 1, 1);
+  }
+#undef OB_TP
   return 6005;
 }
 

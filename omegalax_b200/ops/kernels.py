@@ -25,6 +25,12 @@ def launch_count() -> int:
     return _launches
 
 
+def add_launches(n: int) -> None:
+    """Count the launches of a replayed CUDA graph."""
+    global _launches
+    _launches += n
+
+
 def _call(name, *args):
     global _launches
     _launches += 1

@@ -40,6 +40,20 @@ _SIGS = {
     "ob_gemm_bf16_pair_grouped_wgrad": [P, P, P, P, I, I, I, I, L, L, I, P, P],
     "ob_attn_fwd": [P, P, P, P, P, P, I, I, L, I, I, I, L, L, L, L, F, I, P, P],
     "ob_attn_bwd": [P, P, P, P, P, P, P, P, P, P, P, P, I, I, L, I, I, I, L, L, L, L, L, L, L, F, I, P, P],
+    "ob_attn_fwd_two_part": [P, P, P, P, P, P, I, I, L, I, I, I, I, L, L, L, L, F, P, P],
+    "ob_embed_rows": [P, P, P, I, I, I, I, P, P],
+    "ob_ln_rows": [P, P, P, P, I, I, F, I, P],
+    "ob_relu_sq": [P, P, L, I, P],
+    "ob_soft_cap": [P, L, F, P],
+    "ob_gla_decay": [P, P, L, I, F, I, P],
+    "ob_gla_scan": [P, L, P, P, P, P, P, I, I, I, I, F, I, P],
+    "ob_gla_norm_gate": [P, P, L, P, P, L, I, I, F, I, P],
+    "ob_gla_step": [P, L, P, P, P, P, P, P, I, I, I, I, F, F, F, I, P],
+    "ob_latent_prepare": [P, L, I, P, P, P, P, I, I, P, P, L, L, P, I, I, I, I, I, F, I, P, P],
+    "ob_latent_absorb": [P, L, I, P, P, I, I, I, I, I, I, P],
+    "ob_latent_expand": [P, P, P, I, I, I, I, I, P],
+    "ob_latent_attn_any": [P, P, L, I, P, L, P, P, P, I, I, P, I, I, I, I, F, I, P],
+    "ob_latent_decode": [P, P, L, I, P, L, P, P, I, I, P, P, P, I, I, I, I, I, F, P],
     "ob_decode_append": [P, P, P, P, P, P, P, I, I, P, P, P, L, I, I, I, I, F, F, I, P],
     "ob_decode_attn": [P, P, P, P, P, I, I, I, I, I, I, I, F, P, P, P, P],
     "ob_peer_scatter_add": [P, P, I, P, I, I, P],
@@ -170,6 +184,7 @@ def check_status(device=None) -> None:
             raise KernelError(
                 f"kernel reported status code {v & 0xFF} from block {v >> 8} on cuda:{key} "
                 "(1 stage-full wait, 2 stage-empty wait, 3/4 accumulator waits, 5 flag wait, "
+                "6 a token id, position or cache row out of range, "
                 "8 store outside the output in a debug build)"
             )
 

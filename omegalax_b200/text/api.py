@@ -1,9 +1,12 @@
-"""Public API for text-only causal language models (Qwen3, Qwen3.5 text).
+"""Public API for text-only causal language models (Qwen3, Qwen3.5 text, Letitar).
 
     model, cfg = init_model("qwen3-smoke", 0, tp_size=1, fsdp_size=1, dp_size=1)
     hidden, aux = forward(model, token_ids, pad_id, cfg)       # hidden is *before* lm_head
     cache = make_cache(cfg, batch, prompt_len, steps)
     logits, cache, aux = decode(model, cache, token_ids, pad_id, cfg)
+
+    model, cfg = load_model(folder, device="cuda")             # class by config.json
+    new_tokens = generate(model, cfg, prompts, max_new_tokens)
 
 Mirrors omegalax/text/api.py:42-146.
 """
@@ -14,6 +17,10 @@ import dataclasses
 import torch
 
 from ..models import sharding_runtime as _rt
+from ..models.letitar import registry as letitar_registry
+from ..models.letitar.config import is_letitar_config
+from ..models.letitar.model import Letitar
+from ..models.paged_sequences import PagedSequences
 from ..models.qwen3 import registry as qwen3_registry
 from ..models.qwen3.cache import Cache, init_cache
 from ..models.qwen3.model import Qwen3
@@ -49,7 +56,11 @@ def resolve_config(model_or_id):
     q35 = _q35()
     if q35.config.is_supported_qwen3_5_model_id(model_or_id):
         return q35.config.make_config(model_or_id).text_config
+    if letitar_registry.is_supported_letitar_model_id(model_or_id):
+        return letitar_registry.build_config(model_or_id)
     hf_cfg = load_hf_config_from_source(model_or_id)
+    if is_letitar_config(hf_cfg):
+        return letitar_registry.build_config(model_or_id)
     mt = hf_cfg.get("model_type")
     if mt in {"qwen3", "qwen3_moe"}:
         return qwen3_registry.make_config_from_hf(hf_cfg)
@@ -58,7 +69,7 @@ def resolve_config(model_or_id):
     raise ValueError(
         f"Unsupported text model/config source '{model_or_id}'. Supported Qwen3 ids: "
         f"{sorted(set(list_qwen3_dense_model_ids() + list_qwen3_moe_model_ids()))}; supported Qwen3.5 ids: "
-        f"{q35.config.list_supported_qwen3_5_model_ids()}.")
+        f"{q35.config.list_supported_qwen3_5_model_ids()}; Letitar ids: {letitar_registry.list_letitar_model_ids()}.")
 
 
 def align_config_to_mesh(cfg, mesh: Mesh):
@@ -81,6 +92,8 @@ def shard_batch_dict(batch: dict, cfg, mesh: Mesh | None = None, device=None) ->
 def model_class_for(cfg):
     if isinstance(cfg, ModelConfig):
         return Qwen3
+    if isinstance(cfg, letitar_registry.LetitarConfig):
+        return Letitar
     if _is_q35_text(cfg):
         return _q35().model.Qwen3_5ForCausalLM
     raise ValueError(f"Unsupported text config type: {type(cfg)}")
@@ -108,15 +121,33 @@ def forward(model, token_ids_BT, pad_id: int, cfg):
     return model(token_ids_BT, segment_ids, None, 0)
 
 
-def decode(model, cache: Cache, token_ids_BT, pad_id: int, cfg):
-    """One prefill / decode call: logits [B,V] at the last non-pad column, the cache, aux."""
-    if not isinstance(model, Qwen3):
-        raise NotImplementedError("decode is only implemented for Qwen3 text models.")
+def load_model(source, *, device=None, dtype=torch.bfloat16):
+    """Model and config from a folder with config.json and safetensors; the class follows config.json."""
+    cfg = resolve_config(str(source))
+    device = device or ("cuda" if torch.cuda.is_available() else "cpu")
+    if isinstance(cfg, letitar_registry.LetitarConfig):
+        from ..models.letitar.loader import create_letitar_from_safetensors
+
+        return create_letitar_from_safetensors(source, device=device, dtype=dtype), cfg
+    if isinstance(cfg, ModelConfig):
+        from ..models.qwen3.loader import create_qwen3_from_safetensors
+
+        return create_qwen3_from_safetensors(source, device=device, dtype=dtype), cfg
+    raise ValueError(f"no text loader for {type(cfg).__name__}")
+
+
+def decode(model, cache: Cache, token_ids_BT, pad_id: int, cfg, select=None):
+    """One prefill / decode call: logits [B,V] at the last non-pad column, the cache, aux.  With a paged
+    cache, ``select`` (bool [B,T]) asks for the logits of the marked tokens instead, in order."""
+    if not isinstance(model, (Qwen3, Letitar)):
+        raise NotImplementedError("decode is only implemented for Qwen3 and Letitar text models.")
     segment_ids = (token_ids_BT != pad_id).to(torch.int32)
-    if isinstance(cache, PagedKVCache):
-        hidden = model.decode_paged(token_ids_BT, segment_ids, cache)
+    if isinstance(cache, PagedSequences):
+        hidden = model.decode_paged(token_ids_BT, segment_ids, cache, select)
         with torch.no_grad():
-            return model.lm_head(hidden), cache, torch.zeros((), device=hidden.device)
+            return model.logits(hidden), cache, torch.zeros((), device=hidden.device)
+    if select is not None:
+        raise NotImplementedError("logits of chosen tokens need a paged cache")
     nrp = count_right_pads(token_ids_BT, pad_id)
     with torch.no_grad():
         hidden, aux = model(token_ids_BT, segment_ids, cache, nrp)
@@ -133,12 +164,19 @@ def decode(model, cache: Cache, token_ids_BT, pad_id: int, cfg):
 
 
 def make_cache(cfg, batch_size: int, token_len: int, generate_steps: int, dtype=torch.bfloat16, device=None,
-               paged: bool | None = None, page_size: int = 64, tp_size: int = 1):
+               paged: bool | None = None, page_size: int = 64, tp_size: int = 1, num_pages: int | None = None):
     """KV cache for ``decode``.  On CUDA with bf16 (head_dim 128) the paged cache + decode kernels
     are used by default; otherwise the contiguous power-of-two cache of the reference.  With
-    ``tp_size`` > 1 the (contiguous) cache holds this tensor-parallel rank's kv heads."""
+    ``tp_size`` > 1 the (contiguous) cache holds this tensor-parallel rank's kv heads.  Letitar models
+    use a ``HybridCache`` in ``dtype``; ``num_pages`` bounds the pages of a paged cache when the
+    sequences together hold fewer tokens than batch_size full ones."""
+    if isinstance(cfg, letitar_registry.LetitarConfig):
+        if tp_size > 1:
+            raise NotImplementedError("Letitar has no tensor-parallel layout")
+        return Letitar.make_cache_for(cfg, batch_size, token_len + generate_steps, page_size=page_size, num_pages=num_pages,
+                                      dtype=dtype, device=device)
     if not isinstance(cfg, ModelConfig):
-        raise NotImplementedError("Cache is only available for Qwen3 text models.")
+        raise NotImplementedError("Cache is only available for Qwen3 and Letitar text models.")
     if tp_size > 1:
         import dataclasses
 
@@ -150,5 +188,50 @@ def make_cache(cfg, batch_size: int, token_len: int, generate_steps: int, dtype=
         paged = (device is not None and torch.device(device).type == "cuda" and dtype == torch.bfloat16
                  and cfg.head_dim == 128 and (cfg.num_heads // cfg.num_kv_heads) in (1, 2, 4, 8))
     if paged:
-        return PagedKVCache(cfg, batch_size, token_len + generate_steps, page_size=page_size, dtype=dtype, device=device)
+        return PagedKVCache(cfg, batch_size, token_len + generate_steps, page_size=page_size, dtype=dtype, device=device,
+                            num_pages=num_pages)
     return init_cache(cfg, batch_size, token_len, generate_steps, dtype, device)
+
+
+NO_TOKEN = -1      # padding id of batches whose rows may hold any vocabulary id
+
+
+def batch_rows(rows, batch_size: int):
+    """[batch_size, longest] int32 batch with ``rows[b]`` (a list, possibly empty) left-aligned in row b."""
+    out = torch.full((batch_size, max(1, max((len(r) for r in rows), default=1))), NO_TOKEN, dtype=torch.int32)
+    for b, r in enumerate(rows):
+        if len(r):
+            out[b, :len(r)] = torch.as_tensor(r, dtype=torch.int32)
+    return out
+
+
+@torch.no_grad()
+def generate(model, cfg, prompts, max_new_tokens: int, *, eos_id: int | None = None):
+    """Greedy continuation of a batch of prompts (lists of ids, any lengths): one prompt call, then one
+    call per token through ``decode`` and a paged cache.  A finished sequence gives its pages back
+    while the others go on.  Returns one list of new ids per prompt."""
+    B = len(prompts)
+    if B == 0 or any(len(p) == 0 for p in prompts):
+        raise ValueError("every prompt needs at least one token")
+    w = next(model.parameters())
+    cache = make_cache(cfg, B, max(len(p) for p in prompts), max_new_tokens, dtype=w.dtype, device=w.device)
+    if not isinstance(cache, PagedSequences):
+        raise NotImplementedError("generate needs a model with a paged cache (CUDA)")
+    out: list[list[int]] = [[] for _ in range(B)]
+    rows = [list(p) for p in prompts]
+    live = set(range(B)) if max_new_tokens > 0 else set()
+    while live:
+        ids = batch_rows(rows, B)
+        if isinstance(model, Qwen3):
+            ids = ids.to(w.device)
+        logits, cache, _ = decode(model, cache, ids, NO_TOKEN, cfg)
+        best = logits.argmax(-1).tolist()
+        rows = [[] for _ in range(B)]
+        for b in sorted(live):
+            out[b].append(best[b])
+            if len(out[b]) == max_new_tokens or best[b] == eos_id:
+                live.discard(b)
+                cache.free_sequence(b)
+            else:
+                rows[b] = [best[b]]
+    return out
