@@ -162,6 +162,104 @@ class ClockSampler:
                 "samples": len(sm), "reasons": sorted(reasons)}
 
 
+SERVE_PROMPTS = [(1, 8192), (8, 1024), (1, 512)]            # (sequences, tokens each)
+SERVE_DECODE = [(1, 4096), (32, 4096), (128, 1024)]         # (sequences, tokens already cached)
+
+
+def serve_bench(args) -> int:
+    """Throughput of ``text.api.decode`` with a paged cache, random weights and ids: whole prompts from an
+    empty cache, and single-token steps.  Each call is timed with CUDA events around it, so the copy of
+    its token ids to the device is inside; logits stay on the device."""
+    import dataclasses
+
+    import torch
+
+    from omegalax_b200.ops import kernels as K
+    from omegalax_b200.ops import lib
+    from omegalax_b200.text import api as text_api
+
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    steps, warmup = max(args.steps, 1), max(args.warmup, 3)
+    for name in ("letitar-8layer-4096", "Qwen/Qwen3-8B"):
+        cfg = text_api.resolve_config(name)
+        if name.startswith("Qwen"):
+            cfg = dataclasses.replace(cfg, num_layers=8)
+        model, cfg = text_api.init_model(cfg, 0, tp_size=1, fsdp_size=1, dp_size=1, device=dev, dtype=torch.bfloat16)
+        weight_bytes = sum(p.numel() for n, p in model.named_parameters() if "embed" not in n) * 2
+        host_ids = name.startswith("letitar")
+        gen = torch.Generator().manual_seed(0)
+
+        def ids(B, T):
+            t = torch.randint(0, cfg.vocab_size, (B, T), generator=gen, dtype=torch.int32)
+            return t if host_ids else t.to(dev)
+
+        def timed(fn, n, before=lambda: None):
+            ms = 0.0
+            for i in range(warmup + n):
+                before()
+                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                torch.cuda.synchronize()
+                e0.record()
+                fn()
+                e1.record()
+                torch.cuda.synchronize()
+                if i >= warmup:
+                    ms += e0.elapsed_time(e1)
+            return ms / n
+
+        def table(tag, fn):
+            if args.kernel_table:
+                from omegalax_b200.utils import profiling
+
+                with open(args.kernel_table, "a") as f:
+                    f.write(f"\n{name}, {tag}\n\n" + profiling.format_table(profiling.kernel_time_table(fn, top=24)) + "\n")
+
+        result = {"metric": "serve_tokens_per_sec", "model": name, "layers": 8, "dtype": "bf16", "data": "synthetic",
+                  "steps": steps, "warmup": warmup, "weight_gb": weight_bytes / 1e9, "prompt": [], "decode": []}
+        sampler = ClockSampler(0)
+        sampler.start()
+        K.reset_launch_count()
+        for B, T in SERVE_PROMPTS:
+            cache = text_api.make_cache(cfg, B, T, 0, device=dev)
+            t = ids(B, T)
+
+            def empty():
+                for b in range(B):
+                    cache.free_sequence(b)
+
+            def call():
+                text_api.decode(model, cache, t, text_api.NO_TOKEN, cfg)
+
+            ms = timed(call, steps, empty)
+            result["prompt"].append({"batch": B, "tokens": T, "ms": ms, "tokens_per_sec": B * T / ms * 1e3})
+            empty()
+            table(f"prompt {B} x {T}", call)
+            del cache
+        for B, ctx in SERVE_DECODE:
+            n = 8 * steps
+            cache = text_api.make_cache(cfg, B, ctx, n + warmup + 2, device=dev)
+            # cached contents do not matter for the time: reserve and count them instead of running ctx prompts
+            cache.reserve([ctx] * B)
+            cache.advance([ctx] * B)
+            t = ids(B, 1)
+
+            def call():
+                text_api.decode(model, cache, t, text_api.NO_TOKEN, cfg)
+
+            ms = timed(call, n)
+            result["decode"].append({"batch": B, "context": ctx, "ms": ms, "tokens_per_sec": B / ms * 1e3,
+                                     "weights_gbs": weight_bytes / ms / 1e6})
+            table(f"decode {B} x context {ctx}", call)
+            del cache
+        result["gpu_launches"], result["clocks"] = K.launch_count(), sampler.stop()
+        lib.check_status()
+        print(json.dumps(result), flush=True)
+        del model
+        torch.cuda.empty_cache()
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -187,7 +285,12 @@ def main() -> int:
                     help="a2a: token exchange by library all_to_all instead of the peer-memory kernels")
     ap.add_argument("--kernel-table", default=None,
                     help="after the timed regions, trace one more step and write its per-kernel device times here")
+    ap.add_argument("--serve", action="store_true",
+                    help="instead of the training benchmark: prompt and decode throughput of an 8-layer Letitar and of "
+                         "an 8-layer Qwen3-8B (same width, heads and feed-forward arithmetic) on one GPU, one JSON line each")
     args = ap.parse_args()
+    if args.serve:
+        return serve_bench(args)
     if args.impl == "reference":
         return reference_arm(args)
     if args.impl == "torch_baseline":   # read by ops.functional / parallel.engine at call time

@@ -8,7 +8,8 @@
 //
 //   gla_decay_kernel   alpha = sigmoid(z + bias)^(1/tau) in place
 //   gla_scan_kernel    packed sequences: CTA = (32 value columns, head, sequence); a thread owns KT key
-//                      rows x 4 value columns of S; 16 lanes share a value quad and add their partial o
+//                      rows x 4 value columns of S (packed fp32 pairs); 16 lanes share a value quad and
+//                      add their partial o
 //   gla_step_kernel    one token per sequence: decay, state update, read-out, per-head RMS norm and
 //                      silu gate in one launch; one pass over the state in memory
 //   gla_norm_gate_kernel  per-head RMS norm of o, weight, times silu(g)
@@ -19,11 +20,31 @@
 
 namespace ob {
 
-template <typename T>
-__global__ void gla_decay_kernel(float* __restrict__ z, const T* __restrict__ bias, long long n, int C, float inv_tau) {
-  const long long stride = (long long)gridDim.x * blockDim.x;
-  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride)
-    z[i] = expf(log_sigmoid(z[i] + to_f(bias[i % C])) * inv_tau);
+// grid (column quads, rows); a thread keeps its bias quad over the rows it walks.  VEC: C % 4 == 0.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) gla_decay_kernel(float* __restrict__ z, const T* __restrict__ bias, long long N, int C,
+                                                        float inv_tau) {
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4;
+  if (c >= C) return;
+  float b[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) b[i] = c + i < C ? to_f(bias[c + i]) : 0.f;
+#pragma unroll 2
+  for (long long n = blockIdx.y; n < N; n += gridDim.y) {
+    float* p = z + n * C + c;
+    if (VEC) {
+      float4 v = load4(p);
+      v.x = expf(log_sigmoid(v.x + b[0]) * inv_tau);
+      v.y = expf(log_sigmoid(v.y + b[1]) * inv_tau);
+      v.z = expf(log_sigmoid(v.z + b[2]) * inv_tau);
+      v.w = expf(log_sigmoid(v.w + b[3]) * inv_tau);
+      store4(p, v);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (c + i < C) p[i] = expf(log_sigmoid(p[i] + b[i]) * inv_tau);
+    }
+  }
 }
 
 struct GlaScanArgs {
@@ -38,14 +59,61 @@ struct GlaScanArgs {
   float q_scale;
 };
 
-constexpr int kScanTok = 8;     // tokens staged at a time
+// two fp32 values in one 64-bit register pair (packed fp32 arithmetic)
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t pair2(float lo, float hi) {
+  return (uint64_t)__float_as_uint(lo) | ((uint64_t)__float_as_uint(hi) << 32);
+}
+__device__ __forceinline__ float lo2(uint64_t v) { return __uint_as_float((uint32_t)v); }
+__device__ __forceinline__ float hi2(uint64_t v) { return __uint_as_float((uint32_t)(v >> 32)); }
 
-template <typename T, int KT>
+// four consecutive elements as they lie in memory, kept unconverted while they are in flight
+template <typename T>
+struct Raw4;
+template <>
+struct Raw4<bf16> {
+  uint2 u;
+  __device__ __forceinline__ void load(const bf16* p) { u = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ void set(int i, bf16 v) {
+    const uint32_t b = (uint32_t)__bfloat16_as_ushort(v) << (16 * (i & 1));
+    if (i < 2) u.x |= b; else u.y |= b;
+  }
+  __device__ __forceinline__ void zero() { u = make_uint2(0, 0); }
+  __device__ __forceinline__ float4 get() const {
+    const float2 a = unpack_bf16(u.x), b = unpack_bf16(u.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+};
+template <>
+struct Raw4<float> {
+  float4 u;
+  __device__ __forceinline__ void load(const float* p) { u = *reinterpret_cast<const float4*>(p); }
+  __device__ __forceinline__ void set(int i, float v) { (&u.x)[i] = v; }
+  __device__ __forceinline__ void zero() { u = make_float4(0.f, 0.f, 0.f, 0.f); }
+  __device__ __forceinline__ float4 get() const { return u; }
+};
+
+// VEC: K, V, the pitch and every base are multiples of four elements.
+// A thread's state pairs rows (k, k+1) of one value column.  Tokens are staged TC at a time (registers
+// -> the other shared buffer while the current one is walked) and walked four at a time, so that the
+// 16 partial sums of four tokens x four columns leave through one transposing reduction over 16 lanes.
+template <typename T, int KT, bool VEC>
 __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
   constexpr int KP = KT * 16;                 // padded key width
   constexpr int NJ = KT / 4;
-  extern __shared__ float sm[];               // 2 x { a[8][KP], k[8][KP], q[8][KP], v[8][32] }
-  constexpr int kBuf = kScanTok * (3 * KP + 32);
+  constexpr int TC = KT > 8 ? 8 : 16;         // tokens per stage
+  constexpr int QN = TC * KP / 512;           // key quads per thread and stage
+  constexpr int kA = 0, kK = TC * KP, kQ = 2 * TC * KP, kV = 3 * TC * KP, kBuf = 3 * TC * KP + TC * 64;
+  extern __shared__ __align__(16) float sm[]; // 2 x { a[TC][KP], k[TC][KP], q[TC][KP], v[TC][32] doubled }
   const int b = blockIdx.z, h = blockIdx.y, v_base = blockIdx.x * 32;
   const int row0 = p.cu[b], len = p.cu[b + 1] - row0;
   if (len <= 0) return;
@@ -57,115 +125,158 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
   const int q_off = h * K, k_off = HK + h * K, v_off = 2 * HK + h * V;
   float* st = p.state + ((long long)b * p.H + h) * (long long)K * V;
 
-  float S[KT][4];
+  uint64_t S[KT / 2][4];
   const bool fresh = p.history[b] == 0;
 #pragma unroll
-  for (int j = 0; j < NJ; ++j)
+  for (int r = 0; r < KT / 2; ++r) {
+    const int k = (r >> 1) * 64 + kg * 4 + (r & 1) * 2;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int k = j * 64 + kg * 4 + i;
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int v = v_base + vq + c;
-        S[j * 4 + i][c] = (!fresh && k < K && v < V) ? st[(long long)k * V + v] : 0.f;
-      }
+    for (int c = 0; c < 4; ++c) {
+      const int v = v_base + vq + c;
+      const bool in = !fresh && v < V;
+      S[r][c] = pair2(in && k < K ? st[(long long)k * V + v] : 0.f, in && k + 1 < K ? st[(long long)(k + 1) * V + v] : 0.f);
     }
+  }
 
-  float ra[KT], rk[KT], rq[KT], rv[2];
+  float4 ra[QN];
+  Raw4<T> rk[QN], rq[QN], rv;
+  const int vt = tid >> 3, vk = (tid & 7) * 4;            // value quad of this thread: token vt, columns vk ..
+  // Loads are unconditional at clamped places, so that all of a stage are in flight at once; what lies
+  // past the end is replaced when the stage is written: decay 1 and zero key leave the state unchanged.
   auto fetch = [&](int t0) {
 #pragma unroll
-    for (int i = 0; i < KT; ++i) {
-      const int e = tid + i * 128, t = t0 + e / KP, k = e % KP;
-      const bool in = t < len && k < K;
-      const long long r = (long long)t * p.ldp;
-      ra[i] = in ? alpha[(long long)t * HK + k] : 0.f;
-      rk[i] = in ? to_f(proj[r + k_off + k]) : 0.f;
-      rq[i] = in ? to_f(proj[r + q_off + k]) * p.q_scale : 0.f;
-    }
+    for (int i = 0; i < QN; ++i) {
+      const int e = (tid + i * 128) * 4, t = min(t0 + e / KP, len - 1), k = e % KP;
+      const float* ap = alpha + (long long)t * HK;
+      const T* r = proj + (long long)t * p.ldp;
+      if (VEC) {
+        const int kc = min(k, K - 4);
+        ra[i] = *reinterpret_cast<const float4*>(ap + kc);
+        rk[i].load(r + k_off + kc);
+        rq[i].load(r + q_off + kc);
+      } else {
+        rk[i].zero();
+        rq[i].zero();
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int e = tid + i * 128, t = t0 + (e >> 5), v = v_base + (e & 31);
-      rv[i] = (t < len && v < V) ? to_f(proj[(long long)t * p.ldp + v_off + v]) : 0.f;
-    }
-  };
-  auto put = [&](float* buf) {
-#pragma unroll
-    for (int i = 0; i < KT; ++i) {
-      const int e = tid + i * 128;
-      buf[e] = ra[i];
-      buf[kScanTok * KP + e] = rk[i];
-      buf[2 * kScanTok * KP + e] = rq[i];
-    }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) buf[3 * kScanTok * KP + tid + i * 128] = rv[i];
-  };
-
-  const bool hi8 = kg & 8, hi4 = kg & 4;
-  const int my_v = v_base + vq + (hi8 ? 2 : 0) + (hi4 ? 1 : 0);
-  const bool writer = (kg & 3) == 0 && my_v < V;
-  float* o = p.o + ((long long)row0 * p.H + h) * V + my_v;
-  const long long o_stride = (long long)p.H * V;
-
-  fetch(0);
-  put(sm);
-  __syncthreads();
-  int cur = 0;
-  for (int t0 = 0; t0 < len; t0 += kScanTok) {
-    const bool more = t0 + kScanTok < len;
-    if (more) fetch(t0 + kScanTok);
-    const float* buf = sm + cur * kBuf;
-    const int nt = min(kScanTok, len - t0);
-#pragma unroll 2
-    for (int t = 0; t < nt; ++t) {
-      const float4 vv = load4(buf + 3 * kScanTok * KP + t * 32 + vq);
-      float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
-#pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        const int c = t * KP + j * 64 + kg * 4;
-        const float4 a4 = load4(buf + c), k4 = load4(buf + kScanTok * KP + c), q4 = load4(buf + 2 * kScanTok * KP + c);
-        const float aa[4] = {a4.x, a4.y, a4.z, a4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          float* s = S[j * 4 + i];
-          s[0] = fmaf(aa[i], s[0], kk[i] * vv.x); o0 = fmaf(qq[i], s[0], o0);
-          s[1] = fmaf(aa[i], s[1], kk[i] * vv.y); o1 = fmaf(qq[i], s[1], o1);
-          s[2] = fmaf(aa[i], s[2], kk[i] * vv.z); o2 = fmaf(qq[i], s[2], o2);
-          s[3] = fmaf(aa[i], s[3], kk[i] * vv.w); o3 = fmaf(qq[i], s[3], o3);
+        for (int c = 0; c < 4; ++c) {
+          const int kc = min(k + c, K - 1);
+          (&ra[i].x)[c] = ap[kc];
+          rk[i].set(c, r[k_off + kc]);
+          rq[i].set(c, r[q_off + kc]);
         }
       }
-      // sum of four values over 16 lanes: halve the set twice, then two plain exchanges
-      float x0 = hi8 ? o2 : o0, x1 = hi8 ? o3 : o1;
-      x0 += __shfl_xor_sync(0xffffffffu, hi8 ? o0 : o2, 8);
-      x1 += __shfl_xor_sync(0xffffffffu, hi8 ? o1 : o3, 8);
-      float y = hi4 ? x1 : x0;
-      y += __shfl_xor_sync(0xffffffffu, hi4 ? x0 : x1, 4);
-      y += __shfl_xor_sync(0xffffffffu, y, 2);
-      y += __shfl_xor_sync(0xffffffffu, y, 1);
-      if (writer) o[(long long)(t0 + t) * o_stride] = y;
+    }
+    const T* r = proj + (long long)min(t0 + min(vt, TC - 1), len - 1) * p.ldp + v_off;
+    if (VEC) {
+      rv.load(r + min(v_base + vk, V - 4));
+    } else {
+      rv.zero();
+#pragma unroll
+      for (int c = 0; c < 4; ++c) rv.set(c, r[min(v_base + vk + c, V - 1)]);
+    }
+  };
+  auto put = [&](float* buf, int t0) {
+#pragma unroll
+    for (int i = 0; i < QN; ++i) {
+      const int e = (tid + i * 128) * 4, k = e % KP;
+      const bool in = t0 + e / KP < len;
+      const float4 kk = rk[i].get(), qq = rq[i].get();
+      float4 a = ra[i], x = kk, y = make_float4(qq.x * p.q_scale, qq.y * p.q_scale, qq.z * p.q_scale, qq.w * p.q_scale);
+#pragma unroll
+      for (int c = 0; c < 4; ++c)
+        if (!in || k + c >= K) {
+          (&a.x)[c] = 1.f;
+          (&x.x)[c] = 0.f;
+          (&y.x)[c] = 0.f;
+        }
+      store4(buf + kA + e, a);
+      store4(buf + kK + e, x);
+      store4(buf + kQ + e, y);
+    }
+    if (vt < TC) {      // value columns past the end are computed and never stored
+      const float4 v = rv.get();
+      float* d = buf + kV + vt * 64 + vk * 2;
+      store4(d, make_float4(v.x, v.x, v.y, v.y));
+      store4(d + 4, make_float4(v.z, v.z, v.w, v.w));
+    }
+  };
+
+  // this lane's place in the reduced 4 x 4 block: token (bits 8, 4), column (bits 2, 1)
+  const bool b8 = kg & 8, b4 = kg & 4, b2 = kg & 2, b1 = kg & 1;
+  const int my_t = (b8 ? 2 : 0) + (b4 ? 1 : 0), my_v = v_base + vq + (b2 ? 2 : 0) + (b1 ? 1 : 0);
+  const long long o_stride = (long long)p.H * V;
+  float* o = p.o + ((long long)row0 * p.H + h) * V + my_v + my_t * o_stride;
+  const bool writer = my_v < V;
+
+  fetch(0);
+  put(sm, 0);
+  __syncthreads();
+  int cur = 0;
+  for (int t0 = 0; t0 < len; t0 += TC) {
+    const bool more = t0 + TC < len;
+    if (more) fetch(t0 + TC);
+    const float* buf = sm + cur * kBuf;
+#pragma unroll 1
+    for (int tb = 0; tb < TC; tb += 4) {
+      float y[4][4];
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        const ulonglong2 v01 = *reinterpret_cast<const ulonglong2*>(buf + kV + (tb + t) * 64 + vq * 2);
+        const ulonglong2 v23 = *reinterpret_cast<const ulonglong2*>(buf + kV + (tb + t) * 64 + vq * 2 + 4);
+        const uint64_t vv[4] = {v01.x, v01.y, v23.x, v23.y};
+        uint64_t acc[4] = {0, 0, 0, 0};
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const float* c = buf + (tb + t) * KP + j * 64 + kg * 4;
+          const ulonglong2 a2 = *reinterpret_cast<const ulonglong2*>(c + kA), k2 = *reinterpret_cast<const ulonglong2*>(c + kK),
+                           q2 = *reinterpret_cast<const ulonglong2*>(c + kQ);
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            S[2 * j][x] = fma2(a2.x, S[2 * j][x], mul2(k2.x, vv[x]));
+            acc[x] = fma2(q2.x, S[2 * j][x], acc[x]);
+            S[2 * j + 1][x] = fma2(a2.y, S[2 * j + 1][x], mul2(k2.y, vv[x]));
+            acc[x] = fma2(q2.y, S[2 * j + 1][x], acc[x]);
+          }
+        }
+#pragma unroll
+        for (int x = 0; x < 4; ++x) y[t][x] = lo2(acc[x]) + hi2(acc[x]);
+      }
+      float y2[2][4], y3[4], y4[2];
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          y2[t][x] = (b8 ? y[t + 2][x] : y[t][x]) + __shfl_xor_sync(0xffffffffu, b8 ? y[t][x] : y[t + 2][x], 8);
+#pragma unroll
+      for (int x = 0; x < 4; ++x) y3[x] = (b4 ? y2[1][x] : y2[0][x]) + __shfl_xor_sync(0xffffffffu, b4 ? y2[0][x] : y2[1][x], 4);
+#pragma unroll
+      for (int x = 0; x < 2; ++x) y4[x] = (b2 ? y3[x + 2] : y3[x]) + __shfl_xor_sync(0xffffffffu, b2 ? y3[x] : y3[x + 2], 2);
+      const float r = (b1 ? y4[1] : y4[0]) + __shfl_xor_sync(0xffffffffu, b1 ? y4[0] : y4[1], 1);
+      if (writer && t0 + tb + my_t < len) o[(long long)(t0 + tb) * o_stride] = r;
     }
     if (more) {
       cur ^= 1;
-      put(sm + cur * kBuf);     // the other buffer: its readers finished before the last barrier
+      put(sm + cur * kBuf, t0 + TC);     // the other buffer: its readers finished before the last barrier
       __syncthreads();
     }
   }
 #pragma unroll
-  for (int j = 0; j < NJ; ++j)
+  for (int r = 0; r < KT / 2; ++r) {
+    const int k = (r >> 1) * 64 + kg * 4 + (r & 1) * 2;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int k = j * 64 + kg * 4 + i;
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int v = v_base + vq + c;
-        if (k < K && v < V) st[(long long)k * V + v] = S[j * 4 + i][c];
-      }
+    for (int c = 0; c < 4; ++c) {
+      const int v = v_base + vq + c;
+      if (v < V && k < K) st[(long long)k * V + v] = lo2(S[r][c]);
+      if (v < V && k + 1 < K) st[(long long)(k + 1) * V + v] = hi2(S[r][c]);
     }
+  }
 }
 
 // one warp per (row, head)
 template <typename T>
 __global__ void gla_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ g, long long ldg,
-                                     const T* __restrict__ w, T* __restrict__ out, long long rows, int H, int V, float eps) {
+                                     const T* __restrict__ w, T* __restrict__ out, long long rows, int H, int V, float eps,
+                                     bool vec) {
   const int lane = threadIdx.x & 31;
   const long long wid = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   if (wid >= rows * H) return;
@@ -175,6 +286,14 @@ __global__ void gla_norm_gate_kernel(const float* __restrict__ o, const T* __res
   const T* grow = g + n * ldg + (long long)h * V;
   T* dst = out + wid * V;
   float ss = 0.f;
+  if (vec) {     // V = 128: one vector per lane
+    const float4 x = load4(orow + lane * 4), gg = load4(grow + lane * 4), ww = load4(w + lane * 4);
+    ss = (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+    const float r = 1.f / sqrtf(warp_sum(ss) / (float)V + eps);
+    store4(dst + lane * 4, make_float4(x.x * r * ww.x * silu_f(gg.x), x.y * r * ww.y * silu_f(gg.y),
+                                       x.z * r * ww.z * silu_f(gg.z), x.w * r * ww.w * silu_f(gg.w)));
+    return;
+  }
   for (int v = lane; v < V; v += 32) ss += orow[v] * orow[v];
   const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)V + eps);
   for (int v = lane; v < V; v += 32) dst[v] = from_f<T>(orow[v] * rstd * to_f(w[v]) * silu_f(to_f(grow[v])));
@@ -226,26 +345,34 @@ __global__ void __launch_bounds__(256) gla_step_kernel(const GlaStepArgs p) {
 #pragma unroll
       for (int i = 0; i < VW; ++i) { acc[i] = 0.f; vv[i] = sv[c * VW + i]; }
       const int r0 = ncol > 256 ? 0 : r;
-#pragma unroll 8
-      for (int k = r0; k < K; k += R) {
-        float* s = st + (long long)k * V + c * VW;
-        const float a = sa[k], kk = sk[k], qq = sq[k];
-        float x[VW];
+      for (int kb = r0; kb < K; kb += 8 * R) {
+        float x[8][VW];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {      // eight state rows in flight before any arithmetic
+          const float* s = st + (long long)min(kb + u * R, K - 1) * V + c * VW;
+          if (VW == 4) *reinterpret_cast<float4*>(x[u]) = *reinterpret_cast<const float4*>(s);
+          else x[u][0] = s[0];
+        }
         if (fresh) {
 #pragma unroll
-          for (int i = 0; i < VW; ++i) x[i] = 0.f;
-        } else if (VW == 4) {
-          *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(s);
-        } else {
-          x[0] = s[0];
+          for (int u = 0; u < 8; ++u)
+#pragma unroll
+            for (int i = 0; i < VW; ++i) x[u][i] = 0.f;
         }
 #pragma unroll
-        for (int i = 0; i < VW; ++i) {
-          x[i] = fmaf(a, x[i], kk * vv[i]);
-          acc[i] = fmaf(qq, x[i], acc[i]);
+        for (int u = 0; u < 8; ++u) {
+          const int k = kb + u * R;
+          if (k >= K) break;
+          float* s = st + (long long)k * V + c * VW;
+          const float a = sa[k], kk = sk[k], qq = sq[k];
+#pragma unroll
+          for (int i = 0; i < VW; ++i) {
+            x[u][i] = fmaf(a, x[u][i], kk * vv[i]);
+            acc[i] = fmaf(qq, x[u][i], acc[i]);
+          }
+          if (VW == 4) *reinterpret_cast<float4*>(s) = *reinterpret_cast<float4*>(x[u]);
+          else s[0] = x[u][0];
         }
-        if (VW == 4) *reinterpret_cast<float4*>(s) = *reinterpret_cast<float4*>(x);
-        else s[0] = x[0];
       }
 #pragma unroll
       for (int i = 0; i < VW; ++i) part[(ncol > 256 ? 0 : r) * V + c * VW + i] = acc[i];
@@ -265,23 +392,25 @@ __global__ void __launch_bounds__(256) gla_step_kernel(const GlaStepArgs p) {
     out[v] = from_f<T>(part[v] * rstd * to_f(((const T*)p.norm_w)[v]) * silu_f(to_f(g[v])));
 }
 
-template <typename T>
-static int launch_scan(const GlaScanArgs& a, int B, cudaStream_t s) {
-  dim3 grid((a.V + 31) / 32, a.H, B);
-#define OB_SCAN(KT)                                                                    \
-  do {                                                                                 \
-    auto kern = gla_scan_kernel<T, KT>;                                                \
-    constexpr int smem = 2 * kScanTok * (3 * KT * 16 + 32) * 4;                        \
-    OB_ENSURE_DYN_SMEM(kern, smem);                                                    \
-    kern<<<grid, 128, smem, s>>>(a);                                                   \
-  } while (0)
-  if (a.K <= 64) OB_SCAN(4);
-  else if (a.K <= 128) OB_SCAN(8);
-  else if (a.K <= 256) OB_SCAN(16);
-  else return 6005;
-#undef OB_SCAN
+template <typename T, int KT, bool VEC>
+static int run_scan(const GlaScanArgs& a, int B, cudaStream_t s) {
+  constexpr int TC = KT > 8 ? 8 : 16, smem = 2 * (3 * TC * KT * 16 + TC * 64) * 4;
+  auto kern = gla_scan_kernel<T, KT, VEC>;
+  OB_ENSURE_DYN_SMEM(kern, smem);
+  kern<<<dim3((a.V + 31) / 32, a.H, B), 128, smem, s>>>(a);
   OB_CHECK_LAUNCH();
   return 0;
+}
+
+template <typename T>
+static int launch_scan(const GlaScanArgs& a, int B, cudaStream_t s) {
+  const bool vec = !((a.K | a.V | (int)(a.ldp & 3)) & 3) && !(((uintptr_t)a.proj | (uintptr_t)a.alpha) & 15);
+#define OB_SCAN(KT) return vec ? run_scan<T, KT, true>(a, B, s) : run_scan<T, KT, false>(a, B, s)
+  if (a.K <= 64) OB_SCAN(4);
+  if (a.K <= 128) OB_SCAN(8);
+  if (a.K <= 256) OB_SCAN(16);
+#undef OB_SCAN
+  return 6005;
 }
 
 template <typename T>
@@ -305,10 +434,17 @@ extern "C" {
 
 int ob_gla_decay(float* z, const void* bias, long long N, int C, float inv_tau, int fp32, cudaStream_t s) {
   if (N <= 0) return 0;
-  const long long n = N * C, blocks = (n + 255) / 256, cap = (long long)num_sms() * 16;
-  const unsigned grid = (unsigned)(blocks < cap ? blocks : cap);
-  if (fp32) gla_decay_kernel<float><<<grid, 256, 0, s>>>(z, (const float*)bias, n, C, inv_tau);
-  else gla_decay_kernel<bf16><<<grid, 256, 0, s>>>(z, (const bf16*)bias, n, C, inv_tau);
+  const int gx = (C + 1023) / 1024;
+  const long long cap = (long long)num_sms() * 16 / gx + 1;
+  const dim3 grid(gx, (unsigned)(N < cap ? N : cap));
+  const bool vec = C % 4 == 0 && !((uintptr_t)z & 15);
+  if (fp32) {
+    if (vec) gla_decay_kernel<float, true><<<grid, 256, 0, s>>>(z, (const float*)bias, N, C, inv_tau);
+    else gla_decay_kernel<float, false><<<grid, 256, 0, s>>>(z, (const float*)bias, N, C, inv_tau);
+  } else {
+    if (vec) gla_decay_kernel<bf16, true><<<grid, 256, 0, s>>>(z, (const bf16*)bias, N, C, inv_tau);
+    else gla_decay_kernel<bf16, false><<<grid, 256, 0, s>>>(z, (const bf16*)bias, N, C, inv_tau);
+  }
   OB_CHECK_LAUNCH();
   return 0;
 }
@@ -324,10 +460,11 @@ int ob_gla_norm_gate(const float* o, const void* g, long long ldg, const void* w
                      int V, float eps, int fp32, cudaStream_t s) {
   if (rows <= 0) return 0;
   const unsigned grid = (unsigned)((rows * H * 32 + 255) / 256);
+  const bool vec = V == 128 && ldg % 4 == 0 && !(((uintptr_t)g | (uintptr_t)o | (uintptr_t)w) & 15);
   if (fp32)
-    gla_norm_gate_kernel<float><<<grid, 256, 0, s>>>(o, (const float*)g, ldg, (const float*)w, (float*)out, rows, H, V, eps);
+    gla_norm_gate_kernel<float><<<grid, 256, 0, s>>>(o, (const float*)g, ldg, (const float*)w, (float*)out, rows, H, V, eps, vec);
   else
-    gla_norm_gate_kernel<bf16><<<grid, 256, 0, s>>>(o, (const bf16*)g, ldg, (const bf16*)w, (bf16*)out, rows, H, V, eps);
+    gla_norm_gate_kernel<bf16><<<grid, 256, 0, s>>>(o, (const bf16*)g, ldg, (const bf16*)w, (bf16*)out, rows, H, V, eps, vec);
   OB_CHECK_LAUNCH();
   return 0;
 }

@@ -86,62 +86,96 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentPrepArg
 }
 
 // ------------------------------------------------------------------------------------------------ absorb / expand
-// q_lat[n, h, r] = sum_d q[n, h, d] W_uk[h*dim + d, r]; CTA = (128 latent columns, head, 8 queries)
-template <typename T, typename O>
+// q_lat[n, h, r] = sum_d q[n, h, d] W_uk[h*dim + d, r]; CTA = (128 latent columns, head, 8 queries):
+// a lane owns 4 columns, the four warps split the sum over d.  VEC: rank % 4 == 0.
+template <typename T, typename O, bool VEC>
 __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict__ q, long long ldq, int head_stride,
                                                             const T* __restrict__ uk, O* __restrict__ out, int N, int H,
                                                             int dim, int rank) {
-  extern __shared__ float sq[];   // [8][dim]
-  const int h = blockIdx.y, n0 = blockIdx.z * 8, r = blockIdx.x * 128 + threadIdx.x;
-  const int nn = min(8, N - n0);
+  extern __shared__ __align__(16) float sq[];   // [dim][8]
+  __shared__ float part[4][8][128];
+  const int h = blockIdx.y, n0 = blockIdx.z * 8, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int r = blockIdx.x * 128 + lane * 4, nn = min(8, N - n0);
   for (int i = threadIdx.x; i < 8 * dim; i += 128) {
     const int t = i / dim, d = i - t * dim;
-    sq[i] = t < nn ? to_f(q[(long long)(n0 + t) * ldq + (long long)h * head_stride + d]) : 0.f;
+    sq[d * 8 + t] = t < nn ? to_f(q[(long long)(n0 + t) * ldq + (long long)h * head_stride + d]) : 0.f;
   }
   __syncthreads();
-  if (r >= rank) return;
   const T* w = uk + (long long)h * dim * rank + r;
-  float acc[8] = {};
-#pragma unroll 16
-  for (int d = 0; d < dim; ++d) {
-    const float x = to_f(w[(long long)d * rank]);
+  float acc[8][4] = {};
+  if (r < rank) {
+#pragma unroll 8
+    for (int d = warp; d < dim; d += 4) {
+      const T* wd = w + (long long)d * rank;
+      float x[4];
+      if (VEC) {
+        *reinterpret_cast<float4*>(x) = load4(wd);
+      } else {
 #pragma unroll
-    for (int t = 0; t < 8; ++t) acc[t] = fmaf(x, sq[t * dim + d], acc[t]);
+        for (int c = 0; c < 4; ++c) x[c] = r + c < rank ? to_f(wd[c]) : 0.f;
+      }
+      const float4 a = load4(sq + d * 8), b = load4(sq + d * 8 + 4);
+      const float qq[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int t = 0; t < 8; ++t)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) acc[t][c] = fmaf(x[c], qq[t], acc[t][c]);
+    }
   }
 #pragma unroll
-  for (int t = 0; t < 8; ++t)
-    if (t < nn) out[((long long)(n0 + t) * H + h) * rank + r] = from_f<O>(acc[t]);
+  for (int t = 0; t < 8; ++t) store4(&part[warp][t][lane * 4], make_float4(acc[t][0], acc[t][1], acc[t][2], acc[t][3]));
+  __syncthreads();
+  const int rc = blockIdx.x * 128 + threadIdx.x;
+  if (rc >= rank) return;
+  for (int t = 0; t < nn; ++t)
+    out[((long long)(n0 + t) * H + h) * rank + rc] =
+        from_f<O>((part[0][t][threadIdx.x] + part[1][t][threadIdx.x]) + (part[2][t][threadIdx.x] + part[3][t][threadIdx.x]));
 }
 
-// o[n, h, v] = sum_r o_lat[n, h, r] W_uv[h*vdim + v, r]; CTA = (16 value rows, head, 8 queries), a warp per row
-template <typename T>
-__global__ void __launch_bounds__(128) latent_expand_kernel(const float* __restrict__ ol, const T* __restrict__ uv,
+// o[n, h, v] = sum_r o_lat[n, h, r] W_uv[h*vdim + v, r]; CTA = (32 value rows, head, 8 queries), four rows
+// per warp.  VEC: rank % 4 == 0.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) latent_expand_kernel(const float* __restrict__ ol, const T* __restrict__ uv,
                                                             T* __restrict__ out, int N, int H, int vdim, int rank) {
-  extern __shared__ float so[];   // [8][rank]
+  extern __shared__ __align__(16) float so[];   // [8][rank padded to 4]
   const int h = blockIdx.y, n0 = blockIdx.z * 8, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int nn = min(8, N - n0);
-  for (int i = threadIdx.x; i < 8 * rank; i += 128) {
-    const int t = i / rank, r = i - t * rank;
-    so[i] = t < nn ? ol[((long long)(n0 + t) * H + h) * rank + r] : 0.f;
+  const int nn = min(8, N - n0), ld = (rank + 3) & ~3;
+  for (int i = threadIdx.x; i < 8 * ld; i += 256) {
+    const int t = i / ld, r = i - t * ld;
+    so[i] = t < nn && r < rank ? ol[((long long)(n0 + t) * H + h) * rank + r] : 0.f;
   }
   __syncthreads();
-  for (int j = 0; j < 4; ++j) {
-    const int v = blockIdx.x * 16 + warp * 4 + j;
-    if (v >= vdim) return;
-    const T* w = uv + ((long long)h * vdim + v) * rank;
-    float acc[8] = {};
-#pragma unroll 4
-    for (int r = lane; r < rank; r += 32) {
-      const float x = to_f(w[r]);
+  const int v0 = blockIdx.x * 32 + warp * 4;
+  if (v0 >= vdim) return;
+  float acc[4][8] = {};
+#pragma unroll 2
+  for (int r = lane * 4; r < rank; r += 128) {
+    float x[4][4];
 #pragma unroll
-      for (int t = 0; t < 8; ++t) acc[t] = fmaf(x, so[t * rank + r], acc[t]);
+    for (int j = 0; j < 4; ++j) {
+      const T* w = uv + ((long long)h * vdim + min(v0 + j, vdim - 1)) * rank + r;
+      if (VEC) {
+        *reinterpret_cast<float4*>(x[j]) = load4(w);
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) x[j][c] = r + c < rank ? to_f(w[c]) : 0.f;
+      }
     }
 #pragma unroll
     for (int t = 0; t < 8; ++t) {
-      const float s = warp_sum(acc[t]);
-      if (lane == 0 && t < nn) out[((long long)(n0 + t) * H + h) * vdim + v] = from_f<T>(s);
+      const float4 o = load4(so + t * ld + r);
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        acc[j][t] = fmaf(x[j][3], o.w, fmaf(x[j][2], o.z, fmaf(x[j][1], o.y, fmaf(x[j][0], o.x, acc[j][t]))));
     }
   }
+#pragma unroll
+  for (int j = 0; j < 4; ++j)
+#pragma unroll
+    for (int t = 0; t < 8; ++t) {
+      const float s = warp_sum(acc[j][t]);
+      if (lane == 0 && t < nn && v0 + j < vdim) out[((long long)(n0 + t) * H + h) * vdim + v0 + j] = from_f<T>(s);
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ any-size attention
@@ -249,21 +283,22 @@ constexpr int kDecKeys = 64;      // keys per tile
 
 // CTA = (key split, block of 16*MT heads, sequence), 8 warps.  Shared memory: Q [16*MT][LD],
 // two key tiles [64][LD], P [16*MT][72] (bf16), LD = rank_pad + rot_pad + 8 (rank padded to a multiple
-// of 64, rot to one of 16; the padding holds zeros).  Scores: warp w owns 16*MT x 8 keys.  Output:
-// warp w owns rank_pad / 8 = 8 * NT latent columns for all heads of the block, in registers.
+// of 64, rot to one of 16; the padding holds zeros).  Scores: a warp owns one 16-head tile and 8 * MT
+// keys.  Output: warp w owns rank_pad / 8 = 8 * NT latent columns for all heads of the block, in registers.
 template <int MT, int NT>
 __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeArgs p) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int HB = 16 * MT;
   constexpr int RP = 64 * NT;
   constexpr int LDP = kDecKeys + 8;
+  constexpr int KG = 8 / MT;                  // key groups of a tile (warps per head tile)
   const int rotp = (p.rot + 15) & ~15;
   const int LD = RP + rotp + 8;
   bf16* sQ = (bf16*)smem;
   bf16* sK = sQ + HB * LD;                    // two tiles
   bf16* sP = sK + 2 * kDecKeys * LD;
-  float* s_max = (float*)(sP + HB * LDP);     // [8][HB]
-  float* s_sum = s_max + 8 * HB;              // [8][HB]
+  float* s_max = (float*)(sP + HB * LDP);     // [KG][HB]
+  float* s_sum = s_max + KG * HB;             // [KG][HB]
   const int b = blockIdx.z, h0 = blockIdx.y * HB, sp = blockIdx.x;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int len = p.len[b];
@@ -289,13 +324,20 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
   }
   const int* bt = p.table + (long long)b * p.max_blocks;
   const int cv = p.rank >> 3, rv = p.rot >> 3;      // 16-byte vectors per row
+  // lane l (mod 8) knows the cache row of key warp + 8 l of a tile; looked up one tile ahead
+  auto find_rows = [&](int t) {
+    const int k = min(t * kDecKeys + warp + 8 * (lane & 7), len - 1);   // past the end: the last row again (masked below)
+    return bt[k / p.page_size] * p.page_size + k % p.page_size;
+  };
+  int rows = find_rows(t_lo);
   auto load_tile = [&](int t) {
     bf16* dst = sK + (t & 1) * kDecKeys * LD;
-    for (int r = warp; r < kDecKeys; r += 8) {
-      const int k = min(t * kDecKeys + r, len - 1);   // rows past the end repeat the last one (masked below)
-      const long long row = (long long)bt[k / p.page_size] * p.page_size + k % p.page_size;
-      const bf16* src = p.cache + row * p.ldc;
-      const uint32_t d = smem_u32(dst + r * LD);
+    const int now = rows;
+    rows = find_rows(min(t + 1, t_hi - 1));
+#pragma unroll
+    for (int i = 0; i < kDecKeys / 8; ++i) {
+      const bf16* src = p.cache + (long long)__shfl_sync(0xffffffffu, now, i) * p.ldc;
+      const uint32_t d = smem_u32(dst + (warp + 8 * i) * LD);
       for (int v = lane; v < cv + rv; v += 32)
         cp16(d + (v < cv ? v * 16 : (RP + (v - cv) * 8) * 2), src + v * 8);
     }
@@ -311,7 +353,8 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
     *reinterpret_cast<uint4*>(sQ + r * LD + (v < cv ? v * 8 : RP + (v - cv) * 8)) = u;
   }
   float o[MT][NT][4];
-  float m[MT][2], l[MT][2];
+  float m[MT][2], l[2] = {0.f, 0.f};
+  const int mt = warp % MT, kgrp = warp / MT;  // this warp's head tile and key group in the score phase
 #pragma unroll
   for (int i = 0; i < MT; ++i) {
 #pragma unroll
@@ -319,7 +362,6 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
 #pragma unroll
       for (int c = 0; c < 4; ++c) o[i][j][c] = 0.f;
     m[i][0] = m[i][1] = -INFINITY;
-    l[i][0] = l[i][1] = 0.f;
   }
   const int ksteps = (RP + rotp) >> 4;
   const int g = lane >> 2, tq = lane & 3;
@@ -332,51 +374,58 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
     }
     __syncthreads();
     const bf16* kt = sK + (t & 1) * kDecKeys * LD;
-    // scores of 8 keys per warp: two k-steps of the B operand per ldmatrix.x4
-    float s[MT][4];
+    // scores [16 heads][8 * MT keys]: two k-steps per round into separate accumulators
+    float s2[2][MT][4];
 #pragma unroll
-    for (int i = 0; i < MT; ++i)
+    for (int e = 0; e < 2; ++e)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) s[i][c] = 0.f;
-    const uint32_t kb = smem_u32(kt + (warp * 8 + (lane & 7)) * LD + (lane >> 3) * 8);
-    const uint32_t qb = smem_u32(sQ + (lane & 15) * LD + (lane >> 4) * 8);
+      for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) s2[e][i][c] = 0.f;
+    const uint32_t qb = smem_u32(sQ + (mt * 16 + (lane & 15)) * LD + (lane >> 4) * 8);
+    // one ldmatrix.x4 brings 8 keys x 32 channels
+    const uint32_t kb = smem_u32(kt + (kgrp * 8 * MT + (lane & 7)) * LD + (lane >> 3) * 8);
     int k = 0;
+#pragma unroll 2
     for (; k + 1 < ksteps; k += 2) {
-      uint32_t bb[4];
-      ldsm4(bb, kb + k * 32);
+      uint32_t a0[4], a1[4], bb[MT][4];
+      ldsm4(a0, qb + k * 32);
+      ldsm4(a1, qb + k * 32 + 32);
+#pragma unroll
+      for (int i = 0; i < MT; ++i) ldsm4(bb[i], kb + (i * 8 * LD + k * 16) * 2);
 #pragma unroll
       for (int i = 0; i < MT; ++i) {
-        uint32_t a[4];
-        ldsm4(a, qb + (i * 16 * LD + k * 16) * 2);
-        mma16816(s[i], a, bb[0], bb[1]);
-        ldsm4(a, qb + (i * 16 * LD + k * 16 + 16) * 2);
-        mma16816(s[i], a, bb[2], bb[3]);
+        mma16816(s2[0][i], a0, bb[i][0], bb[i][1]);
+        mma16816(s2[1][i], a1, bb[i][2], bb[i][3]);
       }
     }
-    if (k < ksteps) {   // odd count: the upper half of the x4 load would pass the row's end, read it again
-      uint32_t bb[4];
-      const uint32_t kb1 = smem_u32(kt + (warp * 8 + (lane & 7)) * LD + ((lane >> 3) & 1) * 8);
-      ldsm4(bb, kb1 + k * 32);
+    if (k < ksteps) {   // odd count: the upper half of the x4 load would pass the row's end, so it repeats the lower
+      uint32_t a0[4], bb[4];
+      ldsm4(a0, qb + k * 32);
+      const uint32_t kb1 = smem_u32(kt + (kgrp * 8 * MT + (lane & 7)) * LD + ((lane >> 3) & 1) * 8);
 #pragma unroll
       for (int i = 0; i < MT; ++i) {
-        uint32_t a[4];
-        ldsm4(a, qb + (i * 16 * LD + k * 16) * 2);
-        mma16816(s[i], a, bb[0], bb[1]);
+        ldsm4(bb, kb1 + (i * 8 * LD + k * 16) * 2);
+        mma16816(s2[0][i], a0, bb[0], bb[1]);
       }
     }
-    // mask, tile maximum over this warp's 8 keys, then over the warps
-    const int key = t * kDecKeys + warp * 8 + tq * 2;
+    // mask, maximum over this warp's keys, then over the key groups
+    float mine[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int i = 0; i < MT; ++i) {
+      const int key = t * kDecKeys + (kgrp * MT + i) * 8 + tq * 2;
 #pragma unroll
-      for (int c = 0; c < 4; ++c) s[i][c] = key + (c & 1) < len ? s[i][c] * p.scale_log2 : -INFINITY;
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        float mx = fmaxf(s[i][2 * r], s[i][2 * r + 1]);
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        if (tq == 0) s_max[warp * HB + i * 16 + r * 8 + g] = mx;
+      for (int c = 0; c < 4; ++c) {
+        const float x = s2[0][i][c] + s2[1][i][c];
+        s2[0][i][c] = key + (c & 1) < len ? x * p.scale_log2 : -INFINITY;
+        mine[c >> 1] = fmaxf(mine[c >> 1], s2[0][i][c]);
       }
+    }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      mine[r] = fmaxf(mine[r], __shfl_xor_sync(0xffffffffu, mine[r], 1));
+      mine[r] = fmaxf(mine[r], __shfl_xor_sync(0xffffffffu, mine[r], 2));
+      if (tq == 0) s_max[kgrp * HB + mt * 16 + r * 8 + g] = mine[r];
     }
     __syncthreads();
 #pragma unroll
@@ -386,18 +435,25 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
         const int hr = i * 16 + r * 8 + g;
         float mx = m[i][r];
 #pragma unroll
-        for (int w = 0; w < 8; ++w) mx = fmaxf(mx, s_max[w * HB + hr]);   // a tile has at least one visible key
+        for (int w = 0; w < KG; ++w) mx = fmaxf(mx, s_max[w * HB + hr]);   // a tile has at least one visible key
         const float a = fast_exp2(m[i][r] - mx);
         m[i][r] = mx;
-        l[i][r] *= a;
+        if (a != 1.f) {
 #pragma unroll
-        for (int j = 0; j < NT; ++j) {
-          o[i][j][2 * r] *= a;
-          o[i][j][2 * r + 1] *= a;
+          for (int j = 0; j < NT; ++j) {
+            o[i][j][2 * r] *= a;
+            o[i][j][2 * r + 1] *= a;
+          }
         }
-        const float p0 = fast_exp2(s[i][2 * r] - mx), p1 = fast_exp2(s[i][2 * r + 1] - mx);
-        l[i][r] += p0 + p1;      // this lane's keys only; summed at the end
-        *reinterpret_cast<uint32_t*>(sP + hr * LDP + warp * 8 + tq * 2) = pack_bf16(p0, p1);
+        if (i == mt) {
+          l[r] *= a;
+#pragma unroll
+          for (int x = 0; x < MT; ++x) {
+            const float p0 = fast_exp2(s2[0][x][2 * r] - mx), p1 = fast_exp2(s2[0][x][2 * r + 1] - mx);
+            l[r] += p0 + p1;      // this lane's keys only; summed at the end
+            *reinterpret_cast<uint32_t*>(sP + hr * LDP + (kgrp * MT + x) * 8 + tq * 2) = pack_bf16(p0, p1);
+          }
+        }
       }
     __syncthreads();
     // o += P V, V = latent columns of the key tile
@@ -427,16 +483,14 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
     }
     __syncthreads();      // the tile and P are free for the next round
   }
-  // row sums: over the four lanes of a row, then over the warps
+  // row sums: over the four lanes of a row, then over the key groups
 #pragma unroll
-  for (int i = 0; i < MT; ++i)
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      float x = l[i][r];
-      x += __shfl_xor_sync(0xffffffffu, x, 1);
-      x += __shfl_xor_sync(0xffffffffu, x, 2);
-      if (tq == 0) s_sum[warp * HB + i * 16 + r * 8 + g] = x;
-    }
+  for (int r = 0; r < 2; ++r) {
+    float x = l[r];
+    x += __shfl_xor_sync(0xffffffffu, x, 1);
+    x += __shfl_xor_sync(0xffffffffu, x, 2);
+    if (tq == 0) s_sum[kgrp * HB + mt * 16 + r * 8 + g] = x;
+  }
   __syncthreads();
 #pragma unroll
   for (int i = 0; i < MT; ++i)
@@ -446,7 +500,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
       if (h >= p.H) continue;
       if (warp == 0 && tq == 0) {
         float t = 0.f;
-        for (int w = 0; w < 8; ++w) t += s_sum[w * HB + hr];
+        for (int w = 0; w < KG; ++w) t += s_sum[w * HB + hr];
         pml[h * 2] = m[i][r];
         pml[h * 2 + 1] = t;
       }
@@ -458,33 +512,48 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
     }
 }
 
-// out[b, h, :] = sum over splits; CTA = (head, sequence)
+// out[b, h, :] = sum over at most 64 splits; CTA = (head, sequence, 128 columns)
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                              float* __restrict__ out, int H, int rank, int splits) {
+  __shared__ float wgt[64];
   const int h = blockIdx.x, b = blockIdx.y;
-  const float* ml = part_ml + (long long)b * splits * H * 2 + h * 2;
+  const float2* ml = (const float2*)part_ml + (long long)b * splits * H + h;
   const float* po = part_o + (long long)b * splits * H * rank + (long long)h * rank;
-  float m = -INFINITY, l = 0.f;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[(long long)s * H * 2]);
-  for (int s = 0; s < splits; ++s) {
-    const float ms = ml[(long long)s * H * 2];
-    if (ms != -INFINITY) l += ml[(long long)s * H * 2 + 1] * fast_exp2(ms - m);
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    float2 x[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) x[i] = lane + 32 * i < splits ? ml[(long long)(lane + 32 * i) * H] : make_float2(-INFINITY, 0.f);
+    const float m = warp_max(fmaxf(x[0].x, x[1].x));
+    float e[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) e[i] = x[i].x == -INFINITY ? 0.f : fast_exp2(x[i].x - m);
+    const float l = warp_sum(e[0] * x[0].y + e[1] * x[1].y);
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    wgt[lane] = e[0] * inv;
+    wgt[lane + 32] = e[1] * inv;
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int c = threadIdx.x; c < rank; c += 128) {
-    float o = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float ms = ml[(long long)s * H * 2];
-      if (ms != -INFINITY) o += po[(long long)s * H * rank + c] * fast_exp2(ms - m);
+  __syncthreads();
+  const int c = blockIdx.z * 128 + threadIdx.x;
+  if (c >= rank) return;
+  float o = 0.f;
+  for (int s0 = 0; s0 < splits; s0 += 16) {
+    float x[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) x[i] = po[(long long)min(s0 + i, splits - 1) * H * rank + c];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      const float w = s0 + i < splits ? wgt[s0 + i] : 0.f;
+      o += w != 0.f ? x[i] * w : 0.f;      // a split without keys wrote no row
     }
-    out[((long long)b * H + h) * rank + c] = o * inv;
   }
+  out[((long long)b * H + h) * rank + c] = o;
 }
 
 template <int MT, int NT>
 static int launch_decode(const LatentDecodeArgs& a, int B, cudaStream_t s) {
   const int LD = 64 * NT + ((a.rot + 15) & ~15) + 8;
-  const int smem = (16 * MT + 2 * kDecKeys) * LD * 2 + 16 * MT * (kDecKeys + 8) * 2 + 2 * 8 * 16 * MT * 4;
+  const int smem = (16 * MT + 2 * kDecKeys) * LD * 2 + 16 * MT * (kDecKeys + 8) * 2 + 2 * (8 / MT) * 16 * MT * 4;
   if (smem > 227 * 1024) return 6005;
   auto kern = latent_decode_kernel<MT, NT>;
   OB_ENSURE_DYN_SMEM(kern, 227 * 1024);
@@ -536,27 +605,47 @@ int ob_latent_absorb(const void* q, long long ldq, int head_stride, const void* 
                      int rank, int fp32, int out_bf16, cudaStream_t s) {
   if (N <= 0) return 0;
   const int smem = 8 * dim * 4;
-  if (smem > 48 * 1024 || (fp32 && out_bf16)) return 6005;
-  dim3 grid((rank + 127) / 128, H, (N + 7) / 8);
-  if (fp32)
-    latent_absorb_kernel<float, float><<<grid, 128, smem, s>>>((const float*)q, ldq, head_stride, (const float*)uk, (float*)out, N, H, dim, rank);
-  else if (out_bf16)
-    latent_absorb_kernel<bf16, bf16><<<grid, 128, smem, s>>>((const bf16*)q, ldq, head_stride, (const bf16*)uk, (bf16*)out, N, H, dim, rank);
-  else
-    latent_absorb_kernel<bf16, float><<<grid, 128, smem, s>>>((const bf16*)q, ldq, head_stride, (const bf16*)uk, (float*)out, N, H, dim, rank);
-  OB_CHECK_LAUNCH();
+  if (smem > 30 * 1024 || (fp32 && out_bf16)) return 6005;
+  const bool vec = rank % 4 == 0 && !((uintptr_t)uk & 15);
+  for (int n0 = 0; n0 < N; n0 += 8 * 65535) {     // gridDim.z limit
+    const int n = N - n0 < 8 * 65535 ? N - n0 : 8 * 65535;
+    const dim3 grid((rank + 127) / 128, H, (n + 7) / 8);
+    const long long qo = n0 * ldq, oo = (long long)n0 * H * rank;
+#define OB_ABSORB(T, O)                                                                                              \
+  do {                                                                                                               \
+    if (vec) latent_absorb_kernel<T, O, true><<<grid, 128, smem, s>>>((const T*)q + qo, ldq, head_stride, (const T*)uk, (O*)out + oo, n, H, dim, rank); \
+    else latent_absorb_kernel<T, O, false><<<grid, 128, smem, s>>>((const T*)q + qo, ldq, head_stride, (const T*)uk, (O*)out + oo, n, H, dim, rank);    \
+  } while (0)
+    if (fp32) OB_ABSORB(float, float);
+    else if (out_bf16) OB_ABSORB(bf16, bf16);
+    else OB_ABSORB(bf16, float);
+#undef OB_ABSORB
+    OB_CHECK_LAUNCH();
+  }
   return 0;
 }
 
 int ob_latent_expand(const float* o_lat, const void* uv, void* out, int N, int H, int vdim, int rank, int fp32,
                      cudaStream_t s) {
   if (N <= 0) return 0;
-  const int smem = 8 * rank * 4;
+  const int smem = 8 * ((rank + 3) & ~3) * 4;
   if (smem > 48 * 1024) return 6005;
-  dim3 grid((vdim + 15) / 16, H, (N + 7) / 8);
-  if (fp32) latent_expand_kernel<float><<<grid, 128, smem, s>>>(o_lat, (const float*)uv, (float*)out, N, H, vdim, rank);
-  else latent_expand_kernel<bf16><<<grid, 128, smem, s>>>(o_lat, (const bf16*)uv, (bf16*)out, N, H, vdim, rank);
-  OB_CHECK_LAUNCH();
+  const bool vec = rank % 4 == 0 && !((uintptr_t)uv & 15);
+  for (int n0 = 0; n0 < N; n0 += 8 * 65535) {
+    const int n = N - n0 < 8 * 65535 ? N - n0 : 8 * 65535;
+    const dim3 grid((vdim + 31) / 32, H, (n + 7) / 8);
+    const float* ol = o_lat + (long long)n0 * H * rank;
+#define OB_EXPAND(T)                                                                                                 \
+  do {                                                                                                               \
+    T* o = (T*)out + (long long)n0 * H * vdim;                                                                       \
+    if (vec) latent_expand_kernel<T, true><<<grid, 256, smem, s>>>(ol, (const T*)uv, o, n, H, vdim, rank);           \
+    else latent_expand_kernel<T, false><<<grid, 256, smem, s>>>(ol, (const T*)uv, o, n, H, vdim, rank);              \
+  } while (0)
+    if (fp32) OB_EXPAND(float);
+    else OB_EXPAND(bf16);
+#undef OB_EXPAND
+    OB_CHECK_LAUNCH();
+  }
   return 0;
 }
 
@@ -587,13 +676,13 @@ int ob_latent_decode(const void* q_lat, const void* q_rot, long long ldq, int he
                      float* part_ml, float* out, int B, int H, int rank, int rot, int splits, float scale,
                      cudaStream_t s) {
   if (B <= 0) return 0;
-  if ((rank & 7) || (rot & 7) || (ldc & 7) || (ldq & 7) || (head_stride & 7) || splits < 1) return 6001;
+  if ((rank & 7) || (rot & 7) || (ldc & 7) || (ldq & 7) || (head_stride & 7) || splits < 1 || splits > 64) return 6001;
   if ((((uintptr_t)q_lat) | ((uintptr_t)q_rot) | ((uintptr_t)cache)) & 15) return 6002;
   LatentDecodeArgs a = {(const bf16*)q_lat, (const bf16*)q_rot, (const bf16*)cache, len, table, part_o, part_ml, ldq, ldc,
                         head_stride, H, rank, rot, max_blocks, page_size, splits, scale * 1.4426950408889634f};
   const int rc = H <= 16 ? dispatch_decode<1>(a, B, s) : dispatch_decode<2>(a, B, s);
   if (rc) return rc;
-  latent_combine_kernel<<<dim3(H, B), 128, 0, s>>>(part_o, part_ml, out, H, rank, splits);
+  latent_combine_kernel<<<dim3(H, B, (rank + 127) / 128), 128, 0, s>>>(part_o, part_ml, out, H, rank, splits);
   OB_CHECK_LAUNCH();
   return 0;
 }

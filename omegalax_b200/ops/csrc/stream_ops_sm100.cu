@@ -12,13 +12,19 @@ __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restri
   const int n = blockIdx.x;
   const int id = ids[n];
   float* o = out + (long long)n * D;
+  const bool vec = D % 4 == 0;      // rows of both tensors then start on vector boundaries
   if (id < 0 || id >= V) {   // a row without a token (padding of a fixed-size decode batch): zeros
     if (id != -1 && threadIdx.x == 0) atomicCAS(status, 0, OB_ERR_BAD_ARG | (n << 8));
     for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = 0.f;
     return;
   }
   const T* r = table + (long long)id * D;
-  for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = to_f(r[i]);
+  if (vec) {
+#pragma unroll 4
+    for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) store4(o + i, load4(r + i));
+  } else {
+    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = to_f(r[i]);
+  }
 }
 
 // y = (x - mean) / sqrt(var + eps) * w + b with the variance of the deviations (two passes over

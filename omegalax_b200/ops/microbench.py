@@ -7,6 +7,7 @@ flush between timed launches, reported against the measured peaks of the box.
     python -m omegalax_b200.ops.microbench decode --batch 32 --ctx 4096
     python -m omegalax_b200.ops.microbench elementwise --rows 32768 --cols 4096
     python -m omegalax_b200.ops.microbench ce --rows 8192 --vocab 151936
+    python -m omegalax_b200.ops.microbench serving --batch 2 --seq 8192 --ctx 4096
 
 ``--iters 0 --warmup N`` only launches the kernels N times (for a profiler capture of a small
 case); ``--baseline`` also times the library counterpart (cuBLAS / SDPA) for comparison.
@@ -192,15 +193,101 @@ def bench_ce(a, dev, flush):
             rows=M, vocab=V, hidden=D)
 
 
+def bench_serving(a, dev, flush):
+    """The forward-only serving kernels, each next to the training / Qwen3 kernel it resembles."""
+    from . import serving as S
+
+    it = lambda fn: timeit(fn, a.iters, a.warmup, flush)  # noqa: E731
+    rn = lambda *s: torch.randn(*s, device=dev).to(bf16)  # noqa: E731
+    B, T, D, H = a.batch, a.seq, a.cols, a.heads
+    N = B * T
+    # row ops
+    x, w, xb, FF = torch.randn(N, D, device=dev), rn(D), rn(N, D), 4 * D
+    _report("layer norm rows fp32 -> bf16", it(lambda: S.layernorm_rows(x, w, w, 1e-5)), None, N * D * 6.0, rows=N, cols=D)
+    _report("  like: rmsnorm bf16", it(lambda: K.rmsnorm_fwd(xb, w, 1e-5, want_rstd=False)), None, N * D * 4.0)
+    up = rn(N, FF)
+    _report("squared relu", it(lambda: S.relu_squared(up)), None, N * FF * 4.0)
+    _report("  like: swiglu", it(lambda: K.swiglu_fwd(up)), None, N * FF * 3.0)
+    ids = torch.randint(0, 32000, (N,), device=dev, dtype=torch.int32)
+    tab = rn(32000, D)
+    _report("embedding rows fp32", it(lambda: S.embed_rows(ids, tab)), None, N * D * 6.0)
+    _report("  like: embedding bf16", it(lambda: K.embedding_fwd(ids, tab)), None, N * D * 4.0)
+    wq = rn(D, D)
+    _report("projection added to fp32 rows", it(lambda: S.project(xb, wq, into=x)), 2.0 * N * D * D, None)
+    _report("  like: projection + bf16 residual", it(lambda: K.gemm(xb, wq, residual=xb)), 2.0 * N * D * D, None)
+    del x, xb, up, ids, tab, wq
+    # prompt attention: 128 + 64 query/key channels, 128 value channels
+    d1, d2, vd, R = 128, 64, 128, 512
+    q, k2, kv = rn(N, H * (d1 + d2)), rn(N, R + d2), rn(N, H * (d1 + vd))
+    cu = torch.arange(B + 1, device=dev, dtype=torch.int32) * T
+    _report("latent attention, prompt (192 / 128 channels)",
+            it(lambda: S.attn_two_part(q, kv, k2[:, R:], kv[:, H * d1:], cu, T, H, d1, d2, vd, 0.07)),
+            float(B) * T * T * H * (d1 + d2 + vd), None, batch=B, seq=T, heads=H)
+    q8, k8 = rn(N, H, 128), rn(N, a.kv_heads, 128)
+    _report("  like: attention fwd 128 channels", it(lambda: K.attn_fwd(q8, k8, k8, cu, T, 0.09, True, want_lse=False)),
+            2.0 * B * T * T * H * 128, None)
+    proj = rn(N, H * (d1 + d2) + R + d2)
+    pos = (torch.arange(N, device=dev) % T).to(torch.int32)
+    row = torch.arange(N, device=dev, dtype=torch.int32)
+    cos = torch.randn(T, d2 // 2, device=dev)
+    nw, cache, packed = rn(R), rn(N, R + d2), rn(N, R + d2)
+    _report("latent prepare (rotate q and key part, norm, store)",
+            it(lambda: S.latent_prepare(proj, pos, row, cos, cos, H, d1, d2, R, dkv_off=H * (d1 + d2), norm_w=nw, cache=cache, packed=packed, eps=1e-5)),
+            None, N * (2.0 * 2 * H * d2 + 2.0 * 3 * (R + d2)))
+    qkv, one, c3 = rn(N, (H + 2 * a.kv_heads) * 128), rn(128), torch.randn(N, 64, device=dev)
+    _report("  like: qk-norm + rope", it(lambda: K.qknorm_rope_fwd(qkv, one, one, c3, c3, H, a.kv_heads, 128, 128, 1e-6)), None,
+            4.0 * N * (H + a.kv_heads) * 128)
+    del q, k2, kv, q8, k8, proj, cache, packed, qkv, c3
+    # recurrence
+    Kd = V = 128
+    pr, z, bias = rn(N, 2 * H * (Kd + V)), torch.randn(N, H * Kd, device=dev), rn(H * Kd)
+    st, hist = torch.zeros(max(B, a.decode_batch), H, Kd, V, device=dev), torch.zeros(B, dtype=torch.int32, device=dev)
+    alpha = S.gla_decay_(z.clone(), bias, 16.0)
+    _report("gla decay", it(lambda: S.gla_decay_(z, bias, 16.0)), None, 8.0 * N * H * Kd)
+    fl = 6.0 * N * H * Kd * V
+    by = N * H * (2.0 * (2 * Kd + V) + 4.0 * (Kd + V))
+    _report("gla scan", it(lambda: S.gla_scan(pr, alpha, st, cu, hist, H, Kd, V, 0.09)), fl, by, batch=B, seq=T, heads=H)
+    Tg = T - T % 64
+    g4 = [torch.randn(B, Tg, H, 128, device=dev) for _ in range(3)]
+    gb = -torch.rand(B, Tg, H, device=dev)
+    _report("  like: gated delta rule fwd", it(lambda: K.gdn_fwd(g4[0], g4[1] * 0.05, g4[2], gb, gb.exp(), save=False)), None,
+            B * Tg * H * 128 * 16.0)
+    del g4
+    o = S.gla_scan(pr, alpha, st, cu, hist, H, Kd, V, 0.09)
+    _report("gla norm + gate", it(lambda: S.gla_norm_gate(o, pr[:, 2 * H * Kd + H * V:], rn(V), 1e-5)), None, N * H * V * 8.0)
+    o2 = rn(N * H, V)
+    _report("  like: gated rmsnorm", it(lambda: K.gated_rmsnorm_fwd(o2, o2, one, 1e-5)), None, N * H * V * 6.0)
+    del o, o2, pr, z, alpha
+    # decode
+    Bd, ctx, page = a.decode_batch, a.ctx, 64
+    seen = torch.full((Bd,), ctx, dtype=torch.int32, device=dev)
+    pd, zd = rn(Bd, 2 * H * (Kd + V)), torch.randn(Bd, H * Kd, device=dev)
+    _report("gla step", it(lambda: S.gla_step(pd, zd, bias, rn(V), st, seen, H, Kd, V, 0.09, 16.0, 1e-5)), None, 8.0 * Bd * H * Kd * V, batch=Bd)
+    blocks = -(-(ctx + 1) // page)
+    table = torch.randperm(Bd * blocks, device=dev).to(torch.int32).view(Bd, blocks)
+    lat, ql, qd = rn(Bd * blocks * page, R + d2), rn(Bd, H, R), rn(Bd, H * (d1 + d2))
+    _report("latent decode attention", it(lambda: S.latent_decode(ql, qd, d1 + d2, d1, d2, lat, seen, table, page, 0.07)),
+            2.0 * Bd * ctx * H * (2 * R + d2), 2.0 * Bd * ctx * (R + d2), batch=Bd, ctx=ctx, heads=H)
+    kp, vp, qq = rn(Bd * blocks, page, a.kv_heads, 128), rn(Bd * blocks, page, a.kv_heads, 128), rn(Bd, H, 128)
+    _report("  like: paged decode attention", it(lambda: K.decode_attn(qq, kp, vp, table, seen, page, 0.09)), None,
+            4.0 * Bd * ctx * a.kv_heads * 128)
+    uk, ol = rn(H * d1, R), torch.randn(Bd, H, R, device=dev)
+    _report("latent absorb", it(lambda: S.latent_absorb(qd, d1 + d2, uk, H, d1, R, bf16)), None, 2.0 * H * R * (d1 + Bd))
+    _report("latent expand", it(lambda: S.latent_expand(ol, uk, d1)), None, 2.0 * H * R * (d1 + 2 * Bd))
+    xw, ww = rn(Bd, R), rn(H * d1, R)
+    _report("  like: decode projection of as many weights", it(lambda: K.gemm(xw, ww)), None, 2.0 * H * d1 * R)
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "attn", "gdn", "decode", "elementwise", "ce"])
+    ap.add_argument("what", choices=["gemm", "attn", "gdn", "decode", "elementwise", "ce", "serving"])
     ap.add_argument("--m", type=int, default=16384)
     ap.add_argument("--n", type=int, default=6144)
     ap.add_argument("--k", type=int, default=4096)
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--seq", type=int, default=4096)
     ap.add_argument("--ctx", type=int, default=4096)
+    ap.add_argument("--decode-batch", type=int, default=32)
     ap.add_argument("--heads", type=int, default=32)
     ap.add_argument("--kv-heads", type=int, default=8)
     ap.add_argument("--k-heads", type=int, default=16)
@@ -216,7 +303,7 @@ def main():
     torch.cuda.set_device(dev)
     flush = torch.zeros(64 * 1024 * 1024, device=dev) if a.iters > 0 else None
     {"gemm": bench_gemm, "attn": bench_attn, "gdn": bench_gdn, "decode": bench_decode,
-     "elementwise": bench_elementwise, "ce": bench_ce}[a.what](a, dev, flush)
+     "elementwise": bench_elementwise, "ce": bench_ce, "serving": bench_serving}[a.what](a, dev, flush)
     torch.cuda.synchronize()
     lib.check_status()
 

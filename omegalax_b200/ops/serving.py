@@ -223,9 +223,9 @@ def latent_decode_fits(dtype, dim: int, rot: int, rank: int) -> bool:
 
 
 def latent_decode_splits(B: int, H: int, capacity: int) -> int:
-    """Key splits per sequence: about one CTA per SM, at least two 64-key tiles of capacity each."""
-    blocks = B * -(-H // 32)
-    return max(1, min(-(-148 // blocks), capacity // 128, 64))
+    """Key splits per sequence: one wave of CTAs over the SMs, at least one 64-key tile of capacity each."""
+    blocks = B * -(-H // (16 if H <= 16 else 32))
+    return max(1, min(148 // blocks, capacity // 64, 64))
 
 
 def latent_decode(q_lat, q, head_stride: int, dim: int, rot: int, cache, seen, block_table, page_size: int, scale: float,
