@@ -5,6 +5,9 @@ into an object and the objects are linked into ``omegalax_b200/ops/libomegalax_b
 The library exposes plain ``extern "C"`` launchers that take raw device pointers and a
 stream, so it has no dependency on libtorch and builds in seconds; Python binds it with
 ctypes (see ``lib.py``).  nvcc cross-compiles without a GPU.
+
+``GROUPS`` names subsets of the sources that a program can build alone, into a library of their own,
+when it needs only those (a decode program in a fresh checkout).
 """
 from __future__ import annotations
 
@@ -23,6 +26,11 @@ DEBUG_LIB = HERE / "libomegalax_b200_debug.so"
 # debug build: GEMM epilogues check every store against the output's extent and record status 8;
 # bounded waits give up after ~0.2 s so a protocol error surfaces quickly
 DEBUG_FLAGS = ["-DOB_DEBUG_BOUNDS", "-DOB_WAIT_CYCLES=400000000ll"]
+
+GROUPS = {
+    "serving": ("gemm_sm100", "gemm_pair_sm100", "gemm_pair_wide_sm100", "attention_two_part_sm100", "gla_sm100",
+                "latent_attention_sm100", "stream_ops_sm100"),
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -48,17 +56,24 @@ def _digest(paths) -> str:
     return h.hexdigest()
 
 
-def sources():
-    return sorted(CSRC.glob("*.cu"))
+def sources(group: str | None = None):
+    if group is None:
+        return sorted(CSRC.glob("*.cu"))
+    return sorted(CSRC / f"{stem}.cu" for stem in GROUPS[group])
 
 
-def build(force: bool = False, verbose: bool = False, debug: bool = False) -> Path:
+def group_lib(group: str) -> Path:
+    return HERE / f"libomegalax_b200_{group}.so"
+
+
+def build(force: bool = False, verbose: bool = False, debug: bool = False, group: str | None = None) -> Path:
     """Compile (if stale) and return the path of the shared library (``debug``: the variant with
-    in-kernel store checks and short wait budgets, ``libomegalax_b200_debug.so``)."""
-    srcs = sources()
+    in-kernel store checks and short wait budgets, ``libomegalax_b200_debug.so``; ``group``: the
+    library of that subset only)."""
+    srcs = sources(group)
     headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    out_lib = DEBUG_LIB if debug else LIB
-    build_dir = BUILD / "debug" if debug else BUILD
+    out_lib = DEBUG_LIB if debug else LIB if group is None else group_lib(group)
+    build_dir = BUILD / "debug" if debug else BUILD if group is None else BUILD / group
     extra = DEBUG_FLAGS if debug else []
     stamp = build_dir / "stamp.txt"
     want = _digest(srcs + headers) + ("-debug" if debug else "")

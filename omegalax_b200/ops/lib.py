@@ -18,6 +18,7 @@ _DEBUG_LIB = os.environ.get("OMEGALAX_B200_DEBUG", "0") == "1" and os.environ.ge
 LIB_PATH = _HERE / ("libomegalax_b200_debug.so" if _DEBUG_LIB else "libomegalax_b200.so")
 
 _lib = None
+_partial = False      # _lib holds one group of kernels only
 _status = {}
 
 from ctypes import c_uint
@@ -110,11 +111,20 @@ def available() -> bool:
     return LIB_PATH.exists()
 
 
-def load():
-    """Load the shared library (building it first when a compiler is present)."""
-    global _lib
-    if _lib is not None:
+def load(group: str | None = None):
+    """Load the shared library (building it first when a compiler is present).  With ``group``, and
+    no complete library in the tree, only that group of kernels is built and loaded; a later call of a
+    kernel outside the group builds the complete library."""
+    global _lib, _partial
+    if _lib is not None and not (_partial and group is None):
         return _lib
+    if group is not None and not LIB_PATH.exists() and not _DEBUG_LIB:
+        from . import build as _build
+
+        if os.environ.get("OMEGALAX_B200_NO_BUILD") != "1" or _build.group_lib(group).exists():
+            path = _build.build(group=group) if os.environ.get("OMEGALAX_B200_NO_BUILD") != "1" else _build.group_lib(group)
+            _lib, _partial = _bind(ctypes.CDLL(str(path))), True
+            return _lib
     if (not LIB_PATH.exists() or _DEBUG_LIB):     # the debug variant is re-checked against the sources every time
         if os.environ.get("OMEGALAX_B200_NO_BUILD") != "1":
             from . import build as _build
@@ -124,13 +134,16 @@ def load():
         raise KernelError(
             f"{LIB_PATH} is missing: run `python -m omegalax_b200.ops.build` (needs nvcc) first"
         )
-    lib = ctypes.CDLL(str(LIB_PATH))
+    _lib, _partial = _bind(ctypes.CDLL(str(LIB_PATH))), False
+    return _lib
+
+
+def _bind(lib):
     for name, sig in _SIGS.items():
         if hasattr(lib, name):
             fn = getattr(lib, name)
             fn.argtypes = sig
             fn.restype = c_int
-    _lib = lib
     if hasattr(lib, "ob_gemm_pair_tune"):
         lib.ob_gemm_pair_tune.argtypes = [c_int, c_int, c_int]
         lib.ob_gemm_pair_tune.restype = None
@@ -265,7 +278,9 @@ def check_canaries() -> None:
 
 
 def call(name: str, *args) -> None:
-    lib = load()
+    lib = _lib if _lib is not None else load()
+    if _partial and not hasattr(lib, name):
+        lib = load()
     rc = getattr(lib, name)(*args)
     if rc != 0:
         raise KernelError(f"{name} failed with code {rc}")

@@ -86,7 +86,7 @@ def main(argv=None) -> int:
     if a.dtype == "float32" and not isinstance(cfg, api.letitar_registry.LetitarConfig):
         print("this model's paged decode path runs in bfloat16 only", file=sys.stderr)
         return 3
-    lib.load()
+    lib.load("serving" if isinstance(cfg, api.letitar_registry.LetitarConfig) else None)
     torch.cuda.set_device(0)
     model, cfg = api.load_model(a.model, device=torch.device("cuda", 0), dtype=getattr(torch, a.dtype))
     runner = TraceRunner(model, cfg, a.max_tokens)
