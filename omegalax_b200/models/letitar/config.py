@@ -12,7 +12,7 @@ from ..rope_scaling import RotaryConfig, YarnScaling
 from ..shard_config import ShardConfig
 
 ARCHITECTURE = "Letitar"
-DEFAULT_DECAY_RANK = 16      # of random-initialised models; a checkpoint's tensor shape decides otherwise
+DEFAULT_DECAY_RANK = 32      # of random-initialised models; a checkpoint's tensor shape decides otherwise
 
 MixerConfig = GatedLinearAttentionConfig | LatentAttentionConfig
 
@@ -110,17 +110,17 @@ def config_to_hf(cfg: LetitarConfig) -> dict:
 
 
 # ---------------------------------------------------------------------------------------------- presets
-def _gla(heads, dim, vdim, tau=16.0, rank=DEFAULT_DECAY_RANK):
+def _gla(heads, dim, vdim, tau=8.0, rank=DEFAULT_DECAY_RANK):
     return GatedLinearAttentionConfig(heads, dim, vdim, tau, rank)
 
 
 def _latent(heads, dim, rot_dim, vdim, rank, kv_from=None, base=10000.0, factor=8.0, original=4096):
     return LatentAttentionConfig(heads, dim, rot_dim, vdim, rank, (dim + rot_dim) ** -0.5,
-                                 RotaryConfig(rot_dim, base, YarnScaling(factor, original, 32.0, 1.0)), kv_from)
+                                 RotaryConfig(rot_dim, base, YarnScaling(factor, original, 16.0, 1.0)), kv_from)
 
 
 def _preset(vocab, width, ff, mixers) -> LetitarConfig:
-    return LetitarConfig(vocab_size=vocab, width=width, norm_eps=1e-5, logit_softcap=30.0,
+    return LetitarConfig(vocab_size=vocab, width=width, norm_eps=1e-6, logit_softcap=25.0,
                          layers=tuple(LayerConfig(m, DenseMLPConfig(ff)) for m in mixers))
 
 

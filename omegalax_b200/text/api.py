@@ -99,6 +99,11 @@ def model_class_for(cfg):
     raise ValueError(f"Unsupported text config type: {type(cfg)}")
 
 
+def is_inference_only(cfg) -> bool:
+    """The family's kernels have no backward pass."""
+    return isinstance(cfg, letitar_registry.LetitarConfig)
+
+
 def init_model(model_or_id, rng: int = 0, *, tp_size: int | None = None, fsdp_size: int | None = None,
                dp_size: int | None = None, device=None, dtype=None, meta: bool = False):
     """Random-initialise a text model; returns (model, cfg).  ``rng`` is an integer seed.

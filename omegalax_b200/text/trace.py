@@ -2,10 +2,10 @@
 
 Nothing is sampled.  Steps arrive as JSON lines,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["b"]}
+    {"step": 7, "entries": [{"id": "chat", "tokens": [41], "want": [0]}, ...], "end": ["mail"]}
 
 and run as one batch each through ``text.api.decode`` with a paged cache: either every entry starts a
-request, or every entry continues one of the running batch by one token.  Logits of the wanted places
+request, or every entry continues a request of the running batch.  Logits of the wanted places
 go to <out>/<step>.f32 (little-endian fp32 [wanted, vocab]), and ``done <step>`` to standard output.
 """
 from __future__ import annotations

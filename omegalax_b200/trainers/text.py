@@ -68,6 +68,9 @@ class TrainConfig:
 
 
 def init_model(cfg_or_model_id, rng: int = 0, *, tp_size=None, fsdp_size=None, dp_size=None, **kw):
+    cfg_or_model_id = text_api.resolve_config(cfg_or_model_id)
+    if text_api.is_inference_only(cfg_or_model_id):
+        raise NotImplementedError(f"{text_api.model_class_for(cfg_or_model_id).__name__} models are inference only")
     return text_api.init_model(cfg_or_model_id, rng, tp_size=tp_size, fsdp_size=fsdp_size, dp_size=dp_size, **kw)
 
 

@@ -74,11 +74,12 @@ def test_squared_relu_and_soft_cap(dtype, n):
 
 
 @BOTH
-def test_embedding_rows_and_bad_ids(dtype):
-    t = rnd(0, 11, 18, dtype=dtype)
+@pytest.mark.parametrize("D", [18, 24, 1500])
+def test_embedding_rows_and_bad_ids(dtype, D):
+    t = rnd(0, 11, D, dtype=dtype)
     y = S.embed_rows(cu(torch.tensor([10, -1, 0], dtype=i32)), cu(t))
     done()
-    assert torch.equal(y.cpu(), torch.stack([t[10].float(), torch.zeros(18), t[0].float()]))
+    assert torch.equal(y.cpu(), torch.stack([t[10].float(), torch.zeros(D), t[0].float()]))
     S.embed_rows(cu(torch.tensor([11], dtype=i32)), cu(t))     # outside the table: reported, nothing read
     with pytest.raises(lib.KernelError, match="status code 6"):
         lib.check_status()
@@ -117,7 +118,8 @@ def gla_want(proj, z, bias, H, K, V, tau, state=None):
 
 
 @BOTH
-@pytest.mark.parametrize("H,K,V,tau", [(2, 32, 64, 16.0), (3, 20, 36, 1.0), (1, 72, 24, 0.25), (2, 128, 33, 5.0), (1, 200, 5, 300.0)])
+@pytest.mark.parametrize("H,K,V,tau", [(2, 32, 64, 16.0), (3, 20, 36, 1.0), (1, 72, 24, 0.25), (2, 128, 33, 5.0), (1, 200, 5, 300.0), (2, 200, 40, 4.0),
+                                       (2, 128, 128, 1.0)])
 def test_gla_scan_unequal_sequences_and_states(dtype, H, K, V, tau):
     lens = [19, 0, 1, 8, 40]
     B, N = len(lens), sum(lens)
@@ -167,13 +169,14 @@ def test_gla_step_token_by_token(dtype, H, K, V, tau):
 
 
 @BOTH
-def test_gla_norm_gate(dtype):
-    H, V, N = 3, 40, 6
-    o, gate, w = torch.randn(N, H, V, generator=gen(1)), rnd(2, N, H * V + 5, dtype=dtype), rnd(3, V, dtype=dtype)
+@pytest.mark.parametrize("V,off", [(40, 5), (128, 8), (128, 3)])
+def test_gla_norm_gate(dtype, V, off):
+    H, N = 3, 6
+    o, gate, w = torch.randn(N, H, V, generator=gen(1)), rnd(2, N, H * V + off, dtype=dtype), rnd(3, V, dtype=dtype)
     o[2] *= 1e-4                                                      # eps matters
-    y = S.gla_norm_gate(cu(o), cu(gate)[:, 5:], cu(w), 1e-5)
+    y = S.gla_norm_gate(cu(o), cu(gate)[:, off:], cu(w), 1e-5)
     done()
-    g = gate.double()[:, 5:]
+    g = gate.double()[:, off:]
     close(y, O.rms_norm(o.double(), w.double(), 1e-5).reshape(N, -1) * g * torch.sigmoid(g), dtype)
 
 
@@ -338,7 +341,7 @@ def new_cache(model, cfg, B, tokens, page_size=8, **kw):
 
 def logits_close(got, want, dtype):
     want = want.double()
-    err = (got.double() - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
+    err = (got.detach().double() - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
     tol = 3e-5 if dtype == f32 else 0.06
     assert float(err.max()) < tol, (float(err.max()), int(err.argmax()), tol)
 

@@ -67,6 +67,10 @@ def test_registry_and_presets():
     assert big.width == 4096 and big.layers[-1].mixer.kv_from == 4
     with pytest.raises(NotImplementedError):
         api.make_cache(cfg, 1, 8, 8, tp_size=2)
+    from omegalax_b200.trainers import text as trainer
+
+    with pytest.raises(NotImplementedError, match="inference only"):
+        trainer.init_model("letitar-smoke", 0, tp_size=1, fsdp_size=1, dp_size=1)
 
 
 @pytest.mark.parametrize("cfg_dict,rank", [(M.EVEN, 8), (M.ODD, 5)])
