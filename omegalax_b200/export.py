@@ -16,10 +16,11 @@ def _family(obj_cfg):
         from .models.qwen3_vl import params as p
 
         return p.qwen3_vl_to_hf_config_dict, p.export_qwen3_vl_to_safetensors
-    if name == "LetitarConfig":
-        from .models.letitar import params as p
+    from .models import stream_registry
 
-        return lambda cfg: p.config_to_hf(cfg), p.export_letitar_to_safetensors
+    if isinstance(obj_cfg, stream_registry.StreamDecoderConfig):
+        f = stream_registry.family_of(obj_cfg)
+        return f.config_to_hf, f.export
     raise TypeError(f"Unsupported config type for export: {type(obj_cfg)}")
 
 

@@ -1,5 +1,6 @@
 """Letitar: decoder-only models of gated-linear-attention and latent-attention layers."""
-from .config import LetitarConfig, LayerConfig, is_supported_letitar_model_id, make_config, make_config_from_hf
+from .config import LayerConfig, LetitarConfig, make_config_from_hf
 from .model import Letitar
+from .registry import FAMILY
 
-__all__ = ["Letitar", "LetitarConfig", "LayerConfig", "is_supported_letitar_model_id", "make_config", "make_config_from_hf"]
+__all__ = ["FAMILY", "Letitar", "LetitarConfig", "LayerConfig", "make_config_from_hf"]

@@ -4,12 +4,9 @@ from __future__ import annotations
 import dataclasses
 from typing import Any, Mapping
 
-import torch
-
-from ..hf_io import load_hf_config_from_source, safetensors_shapes
 from ..mixers import DenseMLPConfig, GatedLinearAttentionConfig, LatentAttentionConfig
 from ..rope_scaling import RotaryConfig, YarnScaling
-from ..shard_config import ShardConfig
+from ..stream_decoder import StreamDecoderConfig
 
 ARCHITECTURE = "Letitar"
 DEFAULT_DECAY_RANK = 32      # of random-initialised models; a checkpoint's tensor shape decides otherwise
@@ -23,19 +20,9 @@ class LayerConfig:
     mlp: DenseMLPConfig | None
 
 
-@dataclasses.dataclass(frozen=True)
-class LetitarConfig:
-    vocab_size: int
-    width: int
-    norm_eps: float
+@dataclasses.dataclass(frozen=True, kw_only=True)
+class LetitarConfig(StreamDecoderConfig):
     logit_softcap: float
-    layers: tuple[LayerConfig, ...]
-    shd_cfg: ShardConfig = dataclasses.field(default_factory=ShardConfig.default)
-    dtype: Any = torch.bfloat16
-
-    @property
-    def num_layers(self) -> int:
-        return len(self.layers)
 
     def __post_init__(self):
         for i, layer in enumerate(self.layers):
@@ -77,14 +64,10 @@ def _layer(i: int, d: Mapping, shapes: Mapping[str, tuple]) -> LayerConfig:
     return LayerConfig(mixer, mlp)
 
 
-def is_letitar_config(hf_cfg: Mapping) -> bool:
-    return hf_cfg.get("architecture") == ARCHITECTURE
-
-
 def make_config_from_hf(hf_cfg: Mapping[str, Any], shapes: Mapping[str, tuple] | None = None) -> LetitarConfig:
     """Parse a config.json dict.  ``shapes`` (tensor name -> shape of the checkpoint) gives the sizes that
     only the tensors know."""
-    if not is_letitar_config(hf_cfg):
+    if hf_cfg.get("architecture") != ARCHITECTURE:
         raise ValueError(f"not a {ARCHITECTURE} config: architecture is {hf_cfg.get('architecture')!r}")
     return LetitarConfig(
         vocab_size=int(hf_cfg["vocab"]), width=int(hf_cfg["width"]), norm_eps=float(hf_cfg["norm"]["eps"]),
@@ -124,7 +107,7 @@ def _preset(vocab, width, ff, mixers) -> LetitarConfig:
                          layers=tuple(LayerConfig(m, DenseMLPConfig(ff)) for m in mixers))
 
 
-_PRESETS = {
+PRESETS = {
     "letitar-smoke": lambda: _preset(512, 128, 384, [_gla(2, 32, 64), _latent(4, 32, 16, 32, 64), _gla(2, 32, 64),
                                                      _latent(4, 32, 16, 32, 64, kv_from=1)]),
     # layers of production size: 4096 wide, 32 heads, as many multiply-adds in the feed-forward as a
@@ -133,18 +116,3 @@ _PRESETS = {
         _latent(32, 128, 64, 128, 512), _gla(32, 128, 128), _gla(32, 128, 128), _gla(32, 128, 128),
         _latent(32, 128, 64, 128, 512), _gla(32, 128, 128), _gla(32, 128, 128), _latent(32, 128, 64, 128, 512, kv_from=4)]),
 }
-
-
-def list_letitar_model_ids() -> list[str]:
-    return sorted(_PRESETS)
-
-
-def is_supported_letitar_model_id(model_id: str) -> bool:
-    return model_id in _PRESETS
-
-
-def make_config(source: str) -> LetitarConfig:
-    """Preset name or a directory with config.json (and, for sizes only tensors know, model.safetensors)."""
-    if source in _PRESETS:
-        return _PRESETS[source]()
-    return make_config_from_hf(load_hf_config_from_source(source), safetensors_shapes(source))

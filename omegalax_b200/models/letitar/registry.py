@@ -1,18 +1,10 @@
-"""Letitar family registry."""
+"""Letitar family description."""
 from __future__ import annotations
 
-from .config import LetitarConfig, is_supported_letitar_model_id, list_letitar_model_ids, make_config, make_config_from_hf
+from ..stream_decoder import Family
+from .config import ARCHITECTURE, PRESETS, LetitarConfig, config_to_hf, make_config_from_hf
+from .loader import key_rules
+from .model import Letitar
 
-
-def build_config(model_id: str) -> LetitarConfig:
-    return make_config(model_id)
-
-
-def get_model_cls(model_id: str | None = None):
-    from .model import Letitar
-
-    return Letitar
-
-
-__all__ = ["LetitarConfig", "build_config", "get_model_cls", "is_supported_letitar_model_id", "list_letitar_model_ids",
-           "make_config", "make_config_from_hf"]
+FAMILY = Family(architecture=ARCHITECTURE, config_cls=LetitarConfig, config_from_hf=make_config_from_hf, config_to_hf=config_to_hf,
+                key_rules=key_rules, model_cls=Letitar, presets=PRESETS, kernels="latent_serving")

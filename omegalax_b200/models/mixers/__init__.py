@@ -5,10 +5,12 @@ A mixer's config has ``cache_spec()`` (what it keeps per token or per sequence, 
 ``store`` the layer's cache tensor, and the result is added into the fp32 rows x.
 """
 from .batch import TokenBatch
-from .feed_forward import DenseMLPConfig, SquaredReluMLP
+from .feed_forward import DenseMLPConfig, GatedMLP, GatedMLPConfig, MixtureOfExperts, MixtureOfExpertsConfig, SquaredReluMLP
 from .gated_linear_attention import GatedLinearAttention, GatedLinearAttentionConfig
 from .latent_attention import LatentAttention, LatentAttentionConfig
-from .layers import LayerNorm, Projection
+from .layers import LayerNorm, Projection, RMSNorm
+from .window_attention import WindowAttention, WindowAttentionConfig
 
-__all__ = ["TokenBatch", "DenseMLPConfig", "SquaredReluMLP", "GatedLinearAttention", "GatedLinearAttentionConfig",
-           "LatentAttention", "LatentAttentionConfig", "LayerNorm", "Projection"]
+__all__ = ["TokenBatch", "DenseMLPConfig", "GatedMLP", "GatedMLPConfig", "MixtureOfExperts", "MixtureOfExpertsConfig",
+           "SquaredReluMLP", "GatedLinearAttention", "GatedLinearAttentionConfig", "LatentAttention", "LatentAttentionConfig",
+           "LayerNorm", "Projection", "RMSNorm", "WindowAttention", "WindowAttentionConfig"]

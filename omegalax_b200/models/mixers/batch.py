@@ -25,7 +25,7 @@ class TokenBatch:
     fresh: bool                 # every sequence with new tokens starts here
     positions: int              # bound on positions, for the rotary tables
     flat: torch.Tensor          # the buffer the tensors above are slices of
-    packed: dict = dataclasses.field(default_factory=dict)   # layer -> packed latent rows of this call
+    shared: dict = dataclasses.field(default_factory=dict)   # layer -> rows of this call that later layers read
 
     @staticmethod
     def build(cache, tokens: list) -> "TokenBatch":

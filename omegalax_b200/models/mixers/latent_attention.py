@@ -58,14 +58,14 @@ class LatentAttention(nn.Module):
             packed = None
             if expand:
                 packed = torch.empty(N, store.shape[1], dtype=proj.dtype, device=proj.device)
-                batch.packed[self.layer] = packed
+                batch.shared[self.layer] = packed
             S.latent_prepare(proj, batch.pos, batch.row, cos, sin, H, c.dim, c.rot_dim, c.kv_rank, dkv_off=self.q_rows,
                              norm_w=self.latent_norm, cache=store, eps=self.eps, packed=packed)
         else:
             S.latent_prepare(proj, batch.pos, batch.row, cos, sin, H, c.dim, c.rot_dim, c.kv_rank)
         w = self.kv_proj.weight
         if expand:
-            packed = batch.packed.get(self.layer if c.kv_from is None else c.kv_from)
+            packed = batch.shared.get(self.layer if c.kv_from is None else c.kv_from)
             if packed is None:      # the owner's head sizes kept it off this path: read the rows back from its pages
                 packed = store.index_select(0, batch.row.long())
             kv = S.project(packed[:, :c.kv_rank], w)

@@ -1,4 +1,4 @@
-"""Parameter holders of the serving decoders: projections and layer norm on fp32 rows."""
+"""Parameter holders of the serving decoders: projections and norms of fp32 rows."""
 from __future__ import annotations
 
 import math
@@ -36,3 +36,15 @@ class LayerNorm(nn.Module):
 
     def forward(self, x):
         return S.layernorm_rows(x, self.weight, self.bias, self.eps)
+
+
+class RMSNorm(nn.Module):
+    """x / sqrt(mean(x^2) + eps) * weight, fp32 rows in, weight dtype out."""
+
+    def __init__(self, dim: int, eps: float, device=None, dtype=None):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(dim, device=device, dtype=dtype))
+        self.eps = eps
+
+    def forward(self, x):
+        return S.rms_rows(x, self.weight, self.eps)

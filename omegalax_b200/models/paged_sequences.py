@@ -1,8 +1,10 @@
 """Page bookkeeping shared by the decode caches: a free list of fixed-size pages, a block table and a
 length per sequence.  What a page holds (keys and values, latents) is the subclass's business.
 
-``HybridCache`` is the cache of decoders whose layers differ: pages of latents for latent-attention
-layers, one fp32 state per sequence for recurrent layers, and layers that read another layer's pages.
+``HybridCache`` is the cache of decoders whose layers differ: pages of latents or of keys and values for
+attention layers, one fp32 state per sequence for recurrent layers, and layers that read another layer's
+pages.  When every paged layer looks back over a window only, pages that have left the widest window
+return to the allocator while the sequence goes on.
 """
 from __future__ import annotations
 
@@ -39,6 +41,7 @@ class PagedSequences:
         self.block_table_host = torch.full((batch_size, self.max_blocks), -1, dtype=torch.int32)
         self.block_table = torch.zeros(batch_size, self.max_blocks, dtype=torch.int32, device=device)
         self.blocks_held = [0] * batch_size
+        self.blocks_dropped = [0] * batch_size      # leading blocks given back by drop_before
         self.seq_lens_host = [0] * batch_size
         self.seq_lens = torch.zeros(batch_size, dtype=torch.int32, device=device)
 
@@ -66,11 +69,21 @@ class PagedSequences:
             self.seq_lens_host[b] += n
         self.seq_lens.copy_(torch.tensor(self.seq_lens_host, dtype=torch.int32))
 
+    def drop_before(self, b: int, slot: int) -> None:
+        """Give back the pages of sequence b whose slots all lie before ``slot`` and are read no more."""
+        first = min(max(slot, 0) // self.page_size, self.blocks_held[b])
+        if first > self.blocks_dropped[b]:
+            gone = slice(self.blocks_dropped[b], first)
+            self.allocator.release(self.block_table_host[b, gone].tolist())
+            self.block_table_host[b, gone] = -1
+            self.blocks_dropped[b] = first
+
     def free_sequence(self, b: int) -> None:
         pages = self.block_table_host[b][self.block_table_host[b] >= 0].tolist()
         self.allocator.release(pages)
         self.block_table_host[b] = -1
         self.blocks_held[b] = 0
+        self.blocks_dropped[b] = 0
         self.seq_lens_host[b] = 0
         self.seq_lens.copy_(torch.tensor(self.seq_lens_host, dtype=torch.int32))
 
@@ -100,6 +113,19 @@ class LatentPages:
 
 
 @dataclasses.dataclass(frozen=True)
+class KeyValuePages:
+    """Paged rows of [value | key] per key/value head, of which a query reads the last ``window`` (0: all)."""
+    kv_heads: int
+    dim: int
+    vdim: int
+    window: int = 0
+
+    @property
+    def pitch(self) -> int:
+        return -(-self.kv_heads * (self.dim + self.vdim) // 8) * 8
+
+
+@dataclasses.dataclass(frozen=True)
 class RecurrentState:
     """One fp32 state [heads, key_dim, value_dim] per sequence."""
     heads: int
@@ -115,7 +141,7 @@ class SharedWith:
 
 class HybridCache(PagedSequences):
     """``specs[i]`` says what layer i keeps; ``stores[i]`` is the tensor: [num_pages * page_size, pitch]
-    for latents, [batch, heads, K, V] fp32 for states.  A sequence without tokens starts from a zero
+    for latents or keys and values, [batch, heads, K, V] fp32 for states.  A sequence without tokens starts from a zero
     state whatever its slot held before, so freeing a sequence clears nothing."""
 
     def __init__(self, specs, batch_size: int, max_tokens_per_seq: int, *, page_size: int = 64, dtype=torch.bfloat16,
@@ -124,7 +150,7 @@ class HybridCache(PagedSequences):
         self.dtype = dtype
         self.stores: list[torch.Tensor] = []
         for i, s in enumerate(specs):
-            if isinstance(s, LatentPages):
+            if isinstance(s, (LatentPages, KeyValuePages)):
                 self.stores.append(torch.zeros(self.num_pages * page_size, s.pitch, dtype=dtype, device=device))
             elif isinstance(s, RecurrentState):
                 self.stores.append(torch.zeros(batch_size, s.heads, s.key_dim, s.value_dim, dtype=torch.float32, device=device))
@@ -134,4 +160,13 @@ class HybridCache(PagedSequences):
                 self.stores.append(self.stores[s.layer])
             else:
                 raise TypeError(f"layer {i}: unknown cache spec {s!r}")
+        windows = [getattr(s, "window", 0) for s in specs if not isinstance(s, RecurrentState)]
+        self.horizon = max(windows) if windows and min(windows) > 0 else 0      # 0: every cached token may be read
         self.decode_graph = None     # recorded single-token step (see decode_graph.py)
+
+    def advance(self, new_tokens: list[int]) -> None:
+        super().advance(new_tokens)
+        if self.horizon:
+            for b, n in enumerate(new_tokens):
+                if n:
+                    self.drop_before(b, self.seq_lens_host[b] + 1 - self.horizon)

@@ -27,9 +27,11 @@ DEBUG_LIB = HERE / "libomegalax_b200_debug.so"
 # bounded waits give up after ~0.2 s so a protocol error surfaces quickly
 DEBUG_FLAGS = ["-DOB_DEBUG_BOUNDS", "-DOB_WAIT_CYCLES=400000000ll"]
 
+_GEMM = ("gemm_sm100", "gemm_pair_sm100", "gemm_pair_wide_sm100")
 GROUPS = {
-    "serving": ("gemm_sm100", "gemm_pair_sm100", "gemm_pair_wide_sm100", "attention_two_part_sm100", "gla_sm100",
-                "latent_attention_sm100", "stream_ops_sm100"),
+    "latent_serving": _GEMM + ("attention_two_part_sm100", "gla_sm100", "latent_attention_sm100", "stream_ops_sm100"),
+    "window_serving": _GEMM + ("attention_window_sm100", "moe_route_sm100", "moe_serve_sm100", "stream_ops_sm100",
+                               "window_attention_sm100"),
 }
 
 NVCC_FLAGS = [

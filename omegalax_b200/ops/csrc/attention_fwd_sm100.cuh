@@ -24,6 +24,9 @@
 // channels may come from two tensors: blocks [0, nb1) of Q and K through the first pair of maps, the
 // rest through the second, whose key part is shared by all heads (latent attention: expanded keys
 // plus one rotated part).  Widths that are not multiples of 64 are zero-filled by the TMA boxes.
+//
+// kWindow: a query sees the last p.window keys up to itself (0: all), and each warpgroup walks from the
+// first KV tile one of its rows sees; p.sink adds one logit per head to the softmax denominator.
 #pragma once
 #include "host_utils.h"
 #include "sm100_common.cuh"
@@ -43,6 +46,8 @@ struct AttnFwdArgs {
   float scale_log2;       // softmax scale * log2(e)
   int nb1;                // 64-channel blocks of Q / K read through the first pair of maps
   int vdim;               // value channels that exist (<= 64 * VB)
+  int window;             // kWindow: keys a query sees, 0 for all
+  const bf16* sink;       // kWindow: [H] logits without a value, or null
   int* status;
 };
 
@@ -57,7 +62,7 @@ struct AttnFwdSmem {
   static constexpr int kTotal = kBarOff + 256 + 1024;
 };
 
-template <int QB, int VB, int KST, int VST>
+template <int QB, int VB, int KST, int VST, bool kWindow = false>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQ2,
@@ -91,14 +96,17 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   if (q0 >= seqlen) return;  // uniform for the whole CTA, nothing allocated yet
 
   const int n_kv_total = (seqlen + 127) >> 7;
-  int n_w[2];
+  int n_w[2];      // a warpgroup's KV tiles are lo_w[w] ... n_w[w] - 1
+  int lo_w[2] = {0, 0};
 #pragma unroll
   for (int w = 0; w < 2; ++w) {
     const int qs = q0 + w * 128;
+    if (kWindow && p.window > 0) lo_w[w] = max(0, qs - p.window + 1) >> 7;
     if (qs >= seqlen) n_w[w] = 0;
     else n_w[w] = p.causal ? min(n_kv_total, (qs >> 7) + 1) : n_kv_total;
   }
   const int n = max(n_w[0], n_w[1]);
+  const int j_lo = lo_w[0];        // the first rows see furthest back
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < 2; ++i) {
@@ -144,9 +152,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
       }
       bool ok = true;
-      for (int j = 0; j < n && ok; ++j) {
-        const int sk = j % KST, sv = j % VST;
-        ok = mbar_wait(&k_empty[sk], ((j / KST) & 1) ^ 1, abort_flag, p.status, OB_ERR_WAIT_EMPTY);
+      for (int j = j_lo; j < n && ok; ++j) {
+        const int t = j - j_lo, sk = t % KST, sv = t % VST;
+        ok = mbar_wait(&k_empty[sk], ((t / KST) & 1) ^ 1, abort_flag, p.status, OB_ERR_WAIT_EMPTY);
         if (!ok) break;
         mbar_expect_tx(&k_full[sk], L::kQTile);
 #pragma unroll
@@ -155,7 +163,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           tma_load_3d(smem + L::kKOff + sk * L::kQTile + kb * 16384, first ? &tmK : &tmK2, &k_full[sk],
                       (first ? kb : kb - p.nb1) * 64, first ? g : 0, seq_start + j * 128);
         }
-        ok = mbar_wait(&v_empty[sv], ((j / VST) & 1) ^ 1, abort_flag, p.status, OB_ERR_WAIT_EMPTY);
+        ok = mbar_wait(&v_empty[sv], ((t / VST) & 1) ^ 1, abort_flag, p.status, OB_ERR_WAIT_EMPTY);
         if (!ok) break;
         mbar_expect_tx(&v_full[sv], L::kVTile);
 #pragma unroll
@@ -188,7 +196,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       };
       bool ok = mbar_wait(&k_full[0], 0, abort_flag, p.status, OB_ERR_WAIT_FULL);
       for (int w = 0; w < 2 && ok; ++w) {
-        if (n_w[w] > 0) {
+        if (n_w[w] > 0 && lo_w[w] == j_lo) {
           ok = mbar_wait(&q_full[w], 0, abort_flag, p.status, OB_ERR_WAIT_FULL);
           if (!ok) break;
           tc_fence_after();
@@ -197,24 +205,32 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
       }
       if (ok) umma_commit(&k_empty[0]);
-      for (int j = 0; j < n && ok; ++j) {
-        const int s = j % VST, kn = (j + 1) % KST;     // stage of this V tile and of the next K tile
-        ok = mbar_wait(&v_full[s], (j / VST) & 1, abort_flag, p.status, OB_ERR_WAIT_FULL);
+      for (int j = j_lo; j < n && ok; ++j) {
+        const int t = j - j_lo;
+        const int s = t % VST, kn = (t + 1) % KST;     // stage of this V tile and of the next K tile
+        ok = mbar_wait(&v_full[s], (t / VST) & 1, abort_flag, p.status, OB_ERR_WAIT_FULL);
         if (!ok) break;
         bool k_next_ready = false;
         for (int w = 0; w < 2 && ok; ++w) {
           if (j >= n_w[w]) continue;
-          ok = mbar_wait(&p_ready[w], j & 1, abort_flag, p.status, OB_ERR_WAIT_MISC);
-          if (!ok) break;
-          tc_fence_after();
-          issue_pv(w, s, j == 0);
-          umma_commit(&o_full[w]);
-          if (j + 1 < n_w[w]) {
+          if (j >= lo_w[w]) {
+            ok = mbar_wait(&p_ready[w], (j - lo_w[w]) & 1, abort_flag, p.status, OB_ERR_WAIT_MISC);
+            if (!ok) break;
+            tc_fence_after();
+            issue_pv(w, s, j == lo_w[w]);
+            umma_commit(&o_full[w]);
+          }
+          if (j + 1 >= lo_w[w] && j + 1 < n_w[w]) {
             if (!k_next_ready) {
-              ok = mbar_wait(&k_full[kn], ((j + 1) / KST) & 1, abort_flag, p.status, OB_ERR_WAIT_FULL);
+              ok = mbar_wait(&k_full[kn], ((t + 1) / KST) & 1, abort_flag, p.status, OB_ERR_WAIT_FULL);
               if (!ok) break;
               tc_fence_after();
               k_next_ready = true;
+            }
+            if (j + 1 == lo_w[w]) {      // (kWindow) this warpgroup's first tile
+              ok = mbar_wait(&q_full[w], 0, abort_flag, p.status, OB_ERR_WAIT_FULL);
+              if (!ok) break;
+              tc_fence_after();
             }
             issue_s(w, kn);
             umma_commit(&s_full[w]);
@@ -240,13 +256,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     constexpr float kRescaleLog2 = 8.f;
     float m_ref = -INFINITY, m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
-    const int nj = n_w[w];
-    for (int j = 0; j < nj && ok; ++j) {
-      ok = mbar_wait(&s_full[w], j & 1, abort_flag, p.status, OB_ERR_WAIT_TMEM_FULL);
+    const int nj = n_w[w], lo = lo_w[w];
+    const int kfirst = kWindow && p.window > 0 ? max(0, qpos - p.window + 1) : 0;    // first visible key
+    for (int j = lo; j < nj && ok; ++j) {
+      ok = mbar_wait(&s_full[w], (j - lo) & 1, abort_flag, p.status, OB_ERR_WAIT_TMEM_FULL);
       if (!ok) break;
       tc_fence_after();
       const int kbase = j * 128;
-      const bool need_mask = (kbase + 128 > seqlen) || (p.causal && kbase + 127 > q0 + w * 128);
+      const bool need_mask = (kbase + 128 > seqlen) || (p.causal && kbase + 127 > q0 + w * 128) ||
+                             (kWindow && p.window > 0 && kbase <= q0 + w * 128 + 127 - p.window);
       const int klimit = p.causal ? min(seqlen - 1, qpos) : seqlen - 1;  // last visible key
       // pass 1: row maximum
       float mx = -INFINITY;
@@ -258,7 +276,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         if (need_mask) {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (kbase + c * 32 + i <= klimit) mx = fmaxf(mx, __uint_as_float(v[i]));
+            if (kbase + c * 32 + i <= klimit && (!kWindow || kbase + c * 32 + i >= kfirst)) mx = fmaxf(mx, __uint_as_float(v[i]));
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) mx = fmaxf(mx, __uint_as_float(v[i]));
@@ -271,8 +289,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (__any_sync(0xffffffffu, mine)) {
         const float m_new = mine ? m_run : m_ref;
         const float alpha = (m_ref == -INFINITY) ? 0.f : fast_exp2(m_ref - m_new);   // 1 for rows that keep their reference
-        if (j > 0) {   // O holds the products of the previous tiles: wait for the last of them, then rescale
-          ok = mbar_wait(&o_full[w], (j - 1) & 1, abort_flag, p.status, OB_ERR_WAIT_TMEM_FULL);
+        if (j > lo) {   // O holds the products of the previous tiles: wait for the last of them, then rescale
+          ok = mbar_wait(&o_full[w], (j - 1 - lo) & 1, abort_flag, p.status, OB_ERR_WAIT_TMEM_FULL);
           if (!ok) break;
           tc_fence_after();
 #pragma unroll 1
@@ -303,8 +321,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           float p0 = fast_exp2(__uint_as_float(v[2 * i]) * p.scale_log2 - m_safe);
           float p1 = fast_exp2(__uint_as_float(v[2 * i + 1]) * p.scale_log2 - m_safe);
           if (need_mask) {
-            if (kbase + c * 32 + 2 * i > klimit) p0 = 0.f;
-            if (kbase + c * 32 + 2 * i + 1 > klimit) p1 = 0.f;
+            const int k0 = kbase + c * 32 + 2 * i;
+            if (k0 > klimit || (kWindow && k0 < kfirst)) p0 = 0.f;
+            if (k0 + 1 > klimit || (kWindow && k0 + 1 < kfirst)) p1 = 0.f;
           }
           lsum += p0 + p1;
           pk[i] = pack_bf16(p0, p1);
@@ -320,7 +339,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     // the accumulator of the last tile
     float o_acc[VD];
     if (ok && nj > 0) {
-      ok = mbar_wait(&o_full[w], (nj - 1) & 1, abort_flag, p.status, OB_ERR_WAIT_TMEM_FULL);
+      ok = mbar_wait(&o_full[w], (nj - 1 - lo) & 1, abort_flag, p.status, OB_ERR_WAIT_TMEM_FULL);
       if (ok) {
         tc_fence_after();
 #pragma unroll
@@ -335,6 +354,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       }
     }
     if (ok && nj > 0 && qpos < seqlen) {
+      if (kWindow && p.sink) l_run += fast_exp2(__bfloat162float(p.sink[h]) * 1.4426950408889634f - m_ref);
       const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
       const long long grow = (long long)seq_start + qpos;
       bf16* op = p.out + grow * p.o_row_stride + (long long)h * p.vdim;
@@ -367,12 +387,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   }
 }
 
-template <int QB, int VB, int KST, int VST>
+template <int QB, int VB, int KST, int VST, bool kWindow = false>
 static int run_attn_fwd(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmQ2,
                         const CUtensorMap& tmK2, const AttnFwdArgs& a, int B, int max_seqlen, cudaStream_t stream) {
   using L = AttnFwdSmem<QB, VB, KST, VST>;
   static_assert(L::kTotal <= 227 * 1024, "shared memory");
-  auto kern = attn_fwd_kernel<QB, VB, KST, VST>;
+  auto kern = attn_fwd_kernel<QB, VB, KST, VST, kWindow>;
   OB_ENSURE_DYN_SMEM(kern, L::kTotal);
   dim3 grid((max_seqlen + 255) / 256, a.H, B);
   kern<<<grid, kAttnThreads, L::kTotal, stream>>>(tmQ, tmK, tmV, tmQ2, tmK2, a);

@@ -4,56 +4,60 @@
 // A single-CTA scan turns the counts into segment offsets padded to multiples of 128 rows and
 // a second pass assigns every (token, slot) pair its row in the expert-sorted buffer.  The rows
 // themselves are moved by the dispatch / combine kernels of the expert-parallel path.
+// The sigmoid form scores every expert on its own: it ranks the logits (the scores of large ones
+// round to 1) and takes no softmax.
 #include "host_utils.h"
-#include "sm100_common.cuh"
+#include "serve_common.cuh"
 
 namespace ob {
 
 constexpr int kMaxEPL = 16;   // experts per lane: E <= 512
 constexpr int kMaxTopK = 16;
 
-__global__ void router_topk_kernel(const bf16* __restrict__ logits, float* __restrict__ probs,
+template <typename T, bool kSigmoid>
+__global__ void router_topk_kernel(const T* __restrict__ logits, long long ldl, float* __restrict__ probs,
                                    float* __restrict__ weights, int* __restrict__ idx, int* __restrict__ counts,
                                    long long M, int E, int k, int renorm) {
   const int lane = threadIdx.x & 31;
   const long long row = (blockIdx.x * (long long)blockDim.x + threadIdx.x) >> 5;
   if (row >= M) return;
-  const int epl = E >> 5;
   float v[kMaxEPL];
   float mx = -INFINITY;
 #pragma unroll
   for (int i = 0; i < kMaxEPL; ++i) {
     v[i] = -INFINITY;
-    if (i < epl) {
-      v[i] = __bfloat162float(logits[row * E + lane + 32 * i]);
+    if (lane + 32 * i < E) {
+      v[i] = to_f(logits[row * ldl + lane + 32 * i]);
       mx = fmaxf(mx, v[i]);
     }
   }
-  mx = warp_max(mx);
-  float sum = 0.f;
+  if (!kSigmoid) {
+    mx = warp_max(mx);
+    float sum = 0.f;
 #pragma unroll
-  for (int i = 0; i < kMaxEPL; ++i)
-    if (i < epl) {
-      v[i] = expf(v[i] - mx);
-      sum += v[i];
-    }
-  sum = warp_sum(sum);
-  const float inv = 1.f / sum;
+    for (int i = 0; i < kMaxEPL; ++i)
+      if (lane + 32 * i < E) {
+        v[i] = expf(v[i] - mx);
+        sum += v[i];
+      }
+    sum = warp_sum(sum);
+    const float inv = 1.f / sum;
 #pragma unroll
-  for (int i = 0; i < kMaxEPL; ++i)
-    if (i < epl) {
-      v[i] *= inv;
-      probs[row * E + lane + 32 * i] = v[i];
-    }
+    for (int i = 0; i < kMaxEPL; ++i)
+      if (lane + 32 * i < E) {
+        v[i] *= inv;
+        probs[row * E + lane + 32 * i] = v[i];
+      }
+  }
   float wsel = 0.f;   // lane r keeps the r-th pick
   int isel = 0;
   float tot = 0.f;
   for (int r = 0; r < k; ++r) {
-    float best = -1.f;
+    float best = -INFINITY;
     int bi = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < kMaxEPL; ++i)
-      if (i < epl && v[i] > best) { best = v[i]; bi = lane + 32 * i; }
+      if (lane + 32 * i < E && v[i] > best) { best = v[i]; bi = lane + 32 * i; }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ob_ = __shfl_xor_sync(0xffffffffu, best, o);
@@ -63,11 +67,13 @@ __global__ void router_topk_kernel(const bf16* __restrict__ logits, float* __res
     if ((bi & 31) == lane) {
 #pragma unroll
       for (int i = 0; i < kMaxEPL; ++i)
-        if (i == (bi >> 5)) v[i] = -1.f;   // taken
+        if (i == (bi >> 5)) v[i] = -INFINITY;   // taken
     }
-    if (bi >= E) {  // only with NaN probabilities (no comparison succeeds): keep the ids in range
+    if (bi >= E) {  // only with NaN scores (no comparison succeeds): keep the ids in range
       bi = r;
       best = 0.f;
+    } else if (kSigmoid) {
+      best = 1.f / (1.f + expf(-best));
     }
     if (lane == r) { wsel = best; isel = bi; }
     tot += best;
@@ -233,8 +239,20 @@ int ob_router_topk(const void* logits, float* probs, float* weights, int* idx, i
   if (E % 32 || E > 32 * kMaxEPL || E <= 0) return 6001;
   if (k <= 0 || k > kMaxTopK || k > E) return 6005;
   if (M <= 0) return 0;
-  router_topk_kernel<<<(unsigned)((M * 32 + 255) / 256), 256, 0, s>>>((const bf16*)logits, probs, weights, idx, counts,
-                                                                      M, E, k, renorm);
+  router_topk_kernel<bf16, false><<<(unsigned)((M * 32 + 255) / 256), 256, 0, s>>>((const bf16*)logits, E, probs, weights,
+                                                                                   idx, counts, M, E, k, renorm);
+  OB_CHECK_LAUNCH();
+  return 0;
+}
+
+// fp32 logits [M, E] (pitch ldl) -> the k largest per row: expert ids, and their sigmoids as weights.
+int ob_router_sigmoid_topk(const float* logits, long long ldl, float* weights, int* idx, long long M, int E, int k,
+                           cudaStream_t s) {
+  if (E > 32 * kMaxEPL || E <= 0) return 6001;
+  if (k <= 0 || k > kMaxTopK || k > E) return 6005;
+  if (M <= 0) return 0;
+  router_topk_kernel<float, true><<<(unsigned)((M * 32 + 255) / 256), 256, 0, s>>>(logits, ldl, nullptr, weights, idx, nullptr,
+                                                                                   M, E, k, 0);
   OB_CHECK_LAUNCH();
   return 0;
 }

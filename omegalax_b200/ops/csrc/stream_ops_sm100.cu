@@ -1,6 +1,6 @@
 // Row operations of decoders whose residual stream is kept in fp32: token embedding into fp32 rows,
-// layer norm with bias from fp32 rows to the matrix-product dtype, squared-relu activation,
-// soft-capped logits.  Forward only.  Every kernel exists for bf16 and fp32 weights / outputs.
+// layer norm with bias and RMS norm from fp32 rows to the matrix-product dtype, squared-relu and gated
+// activations, soft-capped logits.  Forward only.  Every kernel exists for bf16 and fp32 weights / outputs.
 #include "host_utils.h"
 #include "serve_common.cuh"
 
@@ -27,11 +27,12 @@ __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restri
   }
 }
 
-// y = (x - mean) / sqrt(var + eps) * w + b with the variance of the deviations (two passes over
-// registers).  One CTA of 256 threads per row; NV float4 per thread cover D <= 1024 * NV, D % 4 == 0.
-template <typename T, int NV>
-__global__ void __launch_bounds__(256) ln_rows_kernel(const float* __restrict__ x, const T* __restrict__ w,
-                                                      const T* __restrict__ b, T* __restrict__ y, int D, float eps) {
+// kMean: y = (x - mean) / sqrt(var + eps) * w + b with the variance of the deviations (two passes over
+// registers); otherwise y = x / sqrt(mean(x^2) + eps) * w.  One CTA of 256 threads per row; NV float4 per
+// thread cover D <= 1024 * NV, D % 4 == 0.
+template <typename T, int NV, bool kMean>
+__global__ void __launch_bounds__(256) norm_rows_kernel(const float* __restrict__ x, const T* __restrict__ w,
+                                                        const T* __restrict__ b, T* __restrict__ y, int D, float eps) {
   __shared__ float red[33];
   const float* xr = x + (long long)blockIdx.x * D;
   T* yr = y + (long long)blockIdx.x * D;
@@ -43,7 +44,7 @@ __global__ void __launch_bounds__(256) ln_rows_kernel(const float* __restrict__ 
     v[i] = c < D ? load4(xr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
   }
-  const float mean = block_sum<256>(s, red) / (float)D;
+  const float mean = kMean ? block_sum<256>(s, red) / (float)D : 0.f;
   float q = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -58,7 +59,7 @@ __global__ void __launch_bounds__(256) ln_rows_kernel(const float* __restrict__ 
   for (int i = 0; i < NV; ++i) {
     const int c = (threadIdx.x + i * 256) * 4;
     if (c < D) {
-      const float4 ww = load4(w + c), bb = load4(b + c);
+      const float4 ww = load4(w + c), bb = kMean ? load4(b + c) : make_float4(0.f, 0.f, 0.f, 0.f);
       store4(yr + c, make_float4(v[i].x * rstd * ww.x + bb.x, v[i].y * rstd * ww.y + bb.y,
                                  v[i].z * rstd * ww.z + bb.z, v[i].w * rstd * ww.w + bb.w));
     }
@@ -66,22 +67,59 @@ __global__ void __launch_bounds__(256) ln_rows_kernel(const float* __restrict__ 
 }
 
 // any D
-template <typename T>
-__global__ void __launch_bounds__(256) ln_rows_any_kernel(const float* __restrict__ x, const T* __restrict__ w,
-                                                          const T* __restrict__ b, T* __restrict__ y, int D, float eps) {
+template <typename T, bool kMean>
+__global__ void __launch_bounds__(256) norm_rows_any_kernel(const float* __restrict__ x, const T* __restrict__ w,
+                                                            const T* __restrict__ b, T* __restrict__ y, int D, float eps) {
   __shared__ float red[33];
   const float* xr = x + (long long)blockIdx.x * D;
   T* yr = y + (long long)blockIdx.x * D;
-  float s = 0.f;
-  for (int c = threadIdx.x; c < D; c += 256) s += xr[c];
-  const float mean = block_sum<256>(s, red) / (float)D;
+  float mean = 0.f;
+  if (kMean) {
+    float s = 0.f;
+    for (int c = threadIdx.x; c < D; c += 256) s += xr[c];
+    mean = block_sum<256>(s, red) / (float)D;
+  }
   float q = 0.f;
   for (int c = threadIdx.x; c < D; c += 256) {
     const float d = xr[c] - mean;
     q += d * d;
   }
   const float rstd = 1.f / sqrtf(block_sum<256>(q, red) / (float)D + eps);
-  for (int c = threadIdx.x; c < D; c += 256) yr[c] = from_f<T>((xr[c] - mean) * rstd * to_f(w[c]) + to_f(b[c]));
+  for (int c = threadIdx.x; c < D; c += 256)
+    yr[c] = from_f<T>((xr[c] - mean) * rstd * to_f(w[c]) + (kMean ? to_f(b[c]) : 0.f));
+}
+
+// act(gate) * up over rows [gate F | up F]; kGelu: the tanh form 0.5 z (1 + tanh t) = z sigmoid(2 t) with
+// t = sqrt(2/pi) (z + 0.044715 z^3), else silu.  bf16 rows take the fast exponential and division.
+template <typename T, bool kGelu>
+__device__ __forceinline__ float gate_value(float z, float up) {
+  const float t = kGelu ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;
+  if (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-t)) * up;
+  return z / (1.f + expf(-t)) * up;
+}
+
+// rows: a device count of the rows that matter (null: all of them).  VEC: F % 8 == 0.
+template <typename T, bool kGelu, bool VEC>
+__global__ void __launch_bounds__(256) gated_act_kernel(const T* __restrict__ x, T* __restrict__ y, const int* __restrict__ rows,
+                                                        long long M, int F) {
+  if (rows) M = min(M, (long long)*rows);
+  const unsigned C = VEC ? F >> 3 : F;
+  const long long n = M * C, stride = (long long)gridDim.x * 256;
+  for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += stride) {
+    const long long r = n < (1ll << 32) ? (unsigned)i / C : i / C;
+    const unsigned c = (unsigned)(i - r * C);
+    const T *a = x + r * 2 * F, *b = a + F;
+    if (VEC) {
+      float g[8], u[8];
+      load8(a + 8 * c, g);
+      load8(b + 8 * c, u);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) g[e] = gate_value<T, kGelu>(g[e], u[e]);
+      store8(y + r * F + 8 * c, g);
+    } else {
+      y[r * F + c] = from_f<T>(gate_value<T, kGelu>(to_f(a[c]), to_f(b[c])));
+    }
+  }
 }
 
 template <typename T>
@@ -106,15 +144,15 @@ __global__ void soft_cap_kernel(float* __restrict__ x, long long n, float cap) {
     x[i] = cap * tanhf(x[i] / cap);
 }
 
-template <typename T>
-static int launch_ln(const float* x, const void* w, const void* b, void* y, int N, int D, float eps, cudaStream_t s) {
+template <typename T, bool kMean>
+static int launch_norm(const float* x, const void* w, const void* b, void* y, int N, int D, float eps, cudaStream_t s) {
   const T *wt = (const T*)w, *bt = (const T*)b;
   T* yt = (T*)y;
-  if (D % 4 || D > 8192) ln_rows_any_kernel<T><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
-  else if (D <= 1024) ln_rows_kernel<T, 1><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
-  else if (D <= 2048) ln_rows_kernel<T, 2><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
-  else if (D <= 4096) ln_rows_kernel<T, 4><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
-  else ln_rows_kernel<T, 8><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
+  if (D % 4 || D > 8192) norm_rows_any_kernel<T, kMean><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
+  else if (D <= 1024) norm_rows_kernel<T, 1, kMean><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
+  else if (D <= 2048) norm_rows_kernel<T, 2, kMean><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
+  else if (D <= 4096) norm_rows_kernel<T, 4, kMean><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
+  else norm_rows_kernel<T, 8, kMean><<<N, 256, 0, s>>>(x, wt, bt, yt, D, eps);
   OB_CHECK_LAUNCH();
   return 0;
 }
@@ -143,7 +181,30 @@ int ob_embed_rows(const int* ids, const void* table, float* out, int N, int V, i
 int ob_ln_rows(const float* x, const void* w, const void* b, void* y, int N, int D, float eps, int fp32,
                cudaStream_t s) {
   if (N <= 0) return 0;
-  return fp32 ? launch_ln<float>(x, w, b, y, N, D, eps, s) : launch_ln<bf16>(x, w, b, y, N, D, eps, s);
+  return fp32 ? launch_norm<float, true>(x, w, b, y, N, D, eps, s) : launch_norm<bf16, true>(x, w, b, y, N, D, eps, s);
+}
+
+int ob_rms_rows(const float* x, const void* w, void* y, int N, int D, float eps, int fp32, cudaStream_t s) {
+  if (N <= 0) return 0;
+  return fp32 ? launch_norm<float, false>(x, w, nullptr, y, N, D, eps, s)
+              : launch_norm<bf16, false>(x, w, nullptr, y, N, D, eps, s);
+}
+
+// x T [M, 2F] = [gate | up] -> y T [M, F]; gelu: 1 tanh-form gelu, 0 silu; rows: device row count or null
+int ob_gated_act(const void* x, void* y, const int* rows, long long M, int F, int gelu, int fp32, cudaStream_t s) {
+  if (M <= 0 || F <= 0) return 0;
+  const bool vec = F % 8 == 0 && !((((uintptr_t)x) | ((uintptr_t)y)) & 15);
+  const unsigned grid = flat_grid(M * (vec ? F / 8 : F));
+#define OB_ACT(T, G)                                                                                  \
+  do {                                                                                                \
+    if (vec) gated_act_kernel<T, G, true><<<grid, 256, 0, s>>>((const T*)x, (T*)y, rows, M, F);       \
+    else gated_act_kernel<T, G, false><<<grid, 256, 0, s>>>((const T*)x, (T*)y, rows, M, F);          \
+  } while (0)
+  if (fp32) { if (gelu) OB_ACT(float, true); else OB_ACT(float, false); }
+  else { if (gelu) OB_ACT(bf16, true); else OB_ACT(bf16, false); }
+#undef OB_ACT
+  OB_CHECK_LAUNCH();
+  return 0;
 }
 
 int ob_relu_sq(const void* x, void* y, long long n, int fp32, cudaStream_t s) {

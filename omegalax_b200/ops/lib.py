@@ -44,7 +44,9 @@ _SIGS = {
     "ob_attn_fwd_two_part": [P, P, P, P, P, P, I, I, L, I, I, I, I, L, L, L, L, F, P, P],
     "ob_embed_rows": [P, P, P, I, I, I, I, P, P],
     "ob_ln_rows": [P, P, P, P, I, I, F, I, P],
+    "ob_rms_rows": [P, P, P, I, I, F, I, P],
     "ob_relu_sq": [P, P, L, I, P],
+    "ob_gated_act": [P, P, P, L, I, I, I, P],
     "ob_soft_cap": [P, L, F, P],
     "ob_gla_decay": [P, P, L, I, F, I, P],
     "ob_gla_scan": [P, L, P, P, P, P, P, I, I, I, I, F, I, P],
@@ -55,6 +57,15 @@ _SIGS = {
     "ob_latent_expand": [P, P, P, I, I, I, I, I, P],
     "ob_latent_attn_any": [P, P, L, I, P, L, P, P, P, I, I, P, I, I, I, I, F, I, P],
     "ob_latent_decode": [P, P, L, I, P, L, P, P, I, I, P, P, P, I, I, I, I, I, F, P],
+    "ob_attn_fwd_window": [P, P, P, P, P, I, I, L, I, I, I, I, L, L, L, F, I, P, P, P],
+    "ob_window_prepare": [P, L, P, P, P, P, I, I, P, P, P, L, P, L, L, I, I, I, I, I, F, I, P, P],
+    "ob_window_attn_any": [P, L, P, L, P, P, P, I, I, P, P, I, I, I, I, I, I, F, I, P],
+    "ob_window_decode": [P, L, P, L, P, P, I, I, P, P, P, P, I, I, I, I, I, I, I, F, P],
+    "ob_router_sigmoid_topk": [P, L, P, P, L, I, I, P],
+    "ob_moe_gather": [P, P, P, P, L, I, I, I, I, P],
+    "ob_moe_sum": [P, P, P, I, I, I, I, I, P],
+    "ob_expert_rows_any": [P, P, P, P, I, I, I, I, I, P],
+    "ob_experts_few": [P, P, P, P, P, P, P, I, I, I, I, I, P],
     "ob_decode_append": [P, P, P, P, P, P, P, I, I, P, P, P, L, I, I, I, I, F, F, I, P],
     "ob_decode_attn": [P, P, P, P, P, I, I, I, I, I, I, I, F, P, P, P, P],
     "ob_peer_scatter_add": [P, P, I, P, I, I, P],

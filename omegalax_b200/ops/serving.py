@@ -1,5 +1,6 @@
-"""Forward-only ops of decoders with an fp32 residual stream: layer norm rows, squared relu, gated
-linear attention, latent attention over a paged latent cache, soft-capped logits.
+"""Forward-only ops of decoders with an fp32 residual stream: norm rows, squared-relu and gated
+activations, gated linear attention, latent attention over a paged latent cache, windowed grouped-query
+attention over paged keys and values, routed experts, soft-capped logits.
 
 Tensors are CUDA bf16 or fp32 (``T`` below: one type per call); the fp32 form of every kernel is
 exact single precision and its matrix products are cuBLAS SGEMMs.  There is no CPU implementation.
@@ -80,6 +81,30 @@ def layernorm_rows(x, w, b, eps: float):
     y = torch.empty(x.shape, dtype=w.dtype, device=x.device)
     K._call("ob_ln_rows", x.data_ptr(), w.data_ptr(), b.data_ptr(), y.data_ptr(), x.shape[0], x.shape[1], float(eps), kind,
             lib.stream_ptr())
+    return y
+
+
+def rms_rows(x, w, eps: float):
+    """fp32 rows -> RMS norm times w, in the dtype of w."""
+    kind = _fp32(w)
+    if x.dtype != f32:
+        raise TypeError("rms_rows reads fp32 rows")
+    _contig(x, w)
+    y = torch.empty(x.shape, dtype=w.dtype, device=x.device)
+    K._call("ob_rms_rows", x.data_ptr(), w.data_ptr(), y.data_ptr(), x.shape[0], x.shape[1], float(eps), kind, lib.stream_ptr())
+    return y
+
+
+GATES = {"silu": 0, "gelu_tanh": 1}
+
+
+def gated_act(gu, act: str, rows=None):
+    """gu [M, 2F] = [gate | up] -> act(gate) * up [M, F].  ``rows`` (int32 [1] on the device): only that
+    many rows hold anything."""
+    _contig(gu)
+    M, F2 = gu.shape
+    y = torch.empty(M, F2 // 2, dtype=gu.dtype, device=gu.device)
+    K._call("ob_gated_act", gu.data_ptr(), y.data_ptr(), lib.ptr(rows), M, F2 // 2, GATES[act], _fp32(gu), lib.stream_ptr())
     return y
 
 
@@ -243,3 +268,147 @@ def latent_decode(q_lat, q, head_stride: int, dim: int, rot: int, cache, seen, b
             cache.data_ptr(), cache.shape[1], seen.data_ptr(), block_table.data_ptr(), block_table.shape[1], page_size,
             part_o.data_ptr(), part_ml.data_ptr(), out.data_ptr(), B, H, rank, rot, splits, float(scale), lib.stream_ptr())
     return out
+
+
+# ----------------------------------------------------------------------------------------------- windowed attention
+def window_prepare(proj, pos, row, cos, sin, H: int, G: int, dim: int, vdim: int, norm_w, cache, eps: float, *, mix=None,
+                   v_first=None):
+    """``proj`` rows [q H*dim | k G*dim | v G*vdim]: norm all of q and all of k, rotate halves by position,
+    mix v with ``v_first`` [N, G*vdim] by the scalar ``mix``; in place, and [v | k] per head into ``cache``
+    [rows, pitch] at ``row``.  ``pos`` -1 marks a row without a token."""
+    kind = _same(proj, norm_w, cache, mix, v_first)
+    _contig(pos, row, cos, sin, norm_w, cache)
+    if (cache.shape[1] < G * (dim + vdim) or norm_w.numel() != (H + G) * dim or proj.shape[1] < (H + G) * dim + G * vdim
+            or proj.stride(1) != 1 or (mix is not None and (v_first is None or v_first.shape[0] < pos.numel()
+                                                            or v_first.shape[1] < G * vdim or v_first.stride(1) != 1))):
+        raise ValueError("projection, norm weights or cache rows do not fit")
+    K._call("ob_window_prepare", proj.data_ptr(), proj.stride(0), pos.data_ptr(), row.data_ptr(), cos.data_ptr(), sin.data_ptr(),
+            cos.shape[0], cos.shape[1], norm_w.data_ptr(), lib.ptr(mix), lib.ptr(v_first),
+            v_first.stride(0) if v_first is not None else 0, cache.data_ptr(), cache.shape[0], cache.shape[1], pos.numel(), H, G,
+            dim, vdim, float(eps), kind, lib.status_tensor(proj.device).data_ptr(), lib.stream_ptr())
+
+
+def window_prompt_fits(dtype, dim: int, vdim: int) -> bool:
+    """Sizes the tcgen05 prompt kernel covers."""
+    return dtype == bf16 and not (dim | vdim) & 7 and dim <= 256 and vdim <= 128
+
+
+def attn_window(q, k, v, cu, max_len: int, H: int, G: int, dim: int, vdim: int, scale: float, window: int, sink=None):
+    """Causal attention over packed rows that all start at position 0: q [N, H*dim], k [N, G*dim],
+    v [N, G*vdim] (row-strided views allowed) -> [N, H*vdim].  A query sees the last ``window`` tokens
+    (0: all); ``sink`` [H] adds a logit without a value to every denominator."""
+    _same(q, k, v, sink)
+    _contig(sink)
+    N = q.shape[0]
+    out = torch.empty(N, H * vdim, dtype=bf16, device=q.device)
+    K._call("ob_attn_fwd_window", q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), cu.data_ptr(), cu.numel() - 1,
+            int(max_len), N, H, G, dim, vdim, q.stride(0), k.stride(0), v.stride(0), float(scale), int(window), lib.ptr(sink),
+            lib.status_tensor(q.device).data_ptr(), lib.stream_ptr())
+    return out
+
+
+def window_attn_any(q, cache, seq, seen, block_table, page_size: int, H: int, G: int, dim: int, vdim: int, scale: float,
+                    window: int, sink=None):
+    """Attention of any query rows against their sequences' cached rows: ``seen`` int32 [N] tokens of
+    sequence ``seq`` end at the query's own.  q [N, H*dim] -> [N, H*vdim]."""
+    kind = _same(q, cache, sink)
+    _contig(cache, seq, seen, block_table, sink)
+    out = torch.empty(q.shape[0], H * vdim, dtype=q.dtype, device=q.device)
+    K._call("ob_window_attn_any", q.data_ptr(), q.stride(0), cache.data_ptr(), cache.shape[1], seq.data_ptr(), seen.data_ptr(),
+            block_table.data_ptr(), block_table.shape[1], page_size, lib.ptr(sink), out.data_ptr(), q.shape[0], H, G, dim, vdim,
+            int(window), float(scale), kind, lib.stream_ptr())
+    return out
+
+
+def window_decode_fits(dtype, dim: int, vdim: int) -> bool:
+    """Sizes the bf16 tensor-core decode kernel covers."""
+    return dtype == bf16 and not (dim | vdim) & 7 and vdim <= 512 and dim + vdim <= 640
+
+
+def window_decode_splits(B: int, H: int, G: int, keys: int) -> int:
+    """Key splits per sequence and key/value head: about two CTAs per SM, at least one 64-key tile each."""
+    R = H // G
+    blocks = B * G * -(-R // (16 if R <= 16 else 32))
+    return max(1, min(296 // blocks, keys // 64, 64))
+
+
+def window_decode(q, cache, seen, block_table, page_size: int, H: int, G: int, dim: int, vdim: int, scale: float, window: int,
+                  sink=None, splits: int | None = None):
+    """One query row per sequence, bf16: q [B, H*dim] -> [B, H*vdim]."""
+    _same(q, cache, sink)
+    _contig(cache, seen, block_table, sink)
+    B = q.shape[0]
+    if splits is None:
+        keys = block_table.shape[1] * page_size
+        splits = window_decode_splits(B, H, G, min(keys, window) if window else keys)
+    part_o = part_ml = None
+    if splits > 1:
+        part_o = torch.empty(B * splits * H * vdim, dtype=f32, device=q.device)
+        part_ml = torch.empty(B * splits * H * 2, dtype=f32, device=q.device)
+    out = torch.empty(B, H * vdim, dtype=bf16, device=q.device)
+    K._call("ob_window_decode", q.data_ptr(), q.stride(0), cache.data_ptr(), cache.shape[1], seen.data_ptr(),
+            block_table.data_ptr(), block_table.shape[1], page_size, lib.ptr(sink), lib.ptr(part_o), lib.ptr(part_ml),
+            out.data_ptr(), B, H, G, dim, vdim, int(window), splits, float(scale), lib.stream_ptr())
+    return out
+
+
+# ----------------------------------------------------------------------------------------------- routed experts
+FEW_PAIRS = 2048      # (token, slot) pairs the kernels without a sort hold
+
+
+def route_sigmoid(logits, top: int):
+    """fp32 logits [M, E] -> (weights fp32 [M, top] = sigmoids of the largest logits, expert ids int32)."""
+    if logits.dtype != f32 or logits.stride(1) != 1:
+        raise TypeError("route_sigmoid reads fp32 rows")
+    M, E = logits.shape
+    w = torch.empty(M, top, dtype=f32, device=logits.device)
+    idx = torch.empty(M, top, dtype=torch.int32, device=logits.device)
+    K._call("ob_router_sigmoid_topk", logits.data_ptr(), logits.stride(0), w.data_ptr(), idx.data_ptr(), M, E, top, lib.stream_ptr())
+    return w, idx
+
+
+def experts_few_fits(dtype, pairs: int, E: int, D: int, F: int) -> bool:
+    """Sizes and counts of the bf16 kernels that stream each expert's weights past the pairs routed to it."""
+    return dtype == bf16 and pairs <= min(FEW_PAIRS, 16 * E) and not (D | F) & 7
+
+
+def experts_into(h, w, idx, gate_up, down, act: str, into, *, few: bool | None = None):
+    """into [M, D] fp32 += sum over the slots of expert(w * h): h T [M, D], w fp32 / idx int32 [M, k],
+    gate_up T [E, 2F, D] with rows [gate | up], down T [E, D, F].  ``few`` overrides the choice of path."""
+    kind = _same(h, gate_up, down)
+    _contig(h, w, idx, gate_up, down, into)
+    (M, k), (E, D, F) = idx.shape, down.shape
+    P, dev = M * k, h.device
+    if gate_up.shape != (E, 2 * F, D) or h.shape != (M, D) or into.shape != (M, D) or into.dtype != f32:
+        raise ValueError("experts, rows or indices do not fit")
+    if P == 0:
+        return into
+    lib.check_index("expert ids", idx, E)
+    fits = act == "silu" and experts_few_fits(h.dtype, P, E, D, F)
+    if fits if few is None else few:
+        mid = torch.empty(P, F, dtype=bf16, device=dev)
+        y = torch.empty(P, D, dtype=f32, device=dev)
+        K._call("ob_experts_few", h.data_ptr(), idx.data_ptr(), w.data_ptr(), gate_up.data_ptr(), down.data_ptr(), mid.data_ptr(),
+                y.data_ptr(), P, k, E, D, F, lib.stream_ptr())
+        K._call("ob_moe_sum", y.data_ptr(), None, into.data_ptr(), M, k, D, P, 1, lib.stream_ptr())
+        return into
+    tiled = not kind and not (D | F) & 7
+    # segments padded to whole tiles; CTA-pair tiles once the experts fill them
+    pad = 1 if not tiled else 256 if P >= 256 * E else 128
+    offsets, dest = K.moe_plan(idx, E, pad)
+    rows = -(-(P + E * (pad - 1)) // pad) * pad
+    xs = torch.empty(rows, D, dtype=h.dtype, device=dev)         # rows between segments stay unwritten and unread
+    K._call("ob_moe_gather", h.data_ptr(), w.data_ptr(), dest.data_ptr(), xs.data_ptr(), P, k, D, rows, kind, lib.stream_ptr())
+    if tiled:
+        gu = K.gemm_grouped(xs, gate_up, offsets, pair=pad == 256)
+        y = K.gemm_grouped(gated_act(gu, act, offsets[E:]), down, offsets, pair=pad == 256)
+    else:
+        def grouped(a, b):
+            out = torch.empty(rows, b.shape[1], dtype=a.dtype, device=dev)
+            K._call("ob_expert_rows_any", a.data_ptr(), b.data_ptr(), out.data_ptr(), offsets.data_ptr(), E, b.shape[1], b.shape[2],
+                    rows, kind, lib.stream_ptr())
+            return out
+
+        y = grouped(gated_act(grouped(xs, gate_up), act, offsets[E:]), down)
+    K._call("ob_moe_sum", y.data_ptr(), dest.data_ptr(), into.data_ptr(), M, k, D, rows, kind, lib.stream_ptr())
+    return into

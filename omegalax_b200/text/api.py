@@ -1,4 +1,5 @@
-"""Public API for text-only causal language models (Qwen3, Qwen3.5 text, Letitar).
+"""Public API for text-only causal language models (Qwen3, Qwen3.5 text, and the serving decoders Letitar
+and Difedra).
 
     model, cfg = init_model("qwen3-smoke", 0, tp_size=1, fsdp_size=1, dp_size=1)
     hidden, aux = forward(model, token_ids, pad_id, cfg)       # hidden is *before* lm_head
@@ -17,9 +18,7 @@ import dataclasses
 import torch
 
 from ..models import sharding_runtime as _rt
-from ..models.letitar import registry as letitar_registry
-from ..models.letitar.config import is_letitar_config
-from ..models.letitar.model import Letitar
+from ..models import stream_registry
 from ..models.paged_sequences import PagedSequences
 from ..models.qwen3 import registry as qwen3_registry
 from ..models.qwen3.cache import Cache, init_cache
@@ -28,6 +27,7 @@ from ..models.qwen3.paged_cache import PagedKVCache
 from ..models.qwen3.utils import count_right_pads
 from ..models.hf_io import load_hf_config_from_source
 from ..models.shard_config import shard_config_for_mesh
+from ..models.stream_decoder import StreamDecoder, StreamDecoderConfig
 from ..parallel.mesh import Mesh, ensure_mesh
 
 ModelConfig = qwen3_registry.Qwen3Config
@@ -56,11 +56,12 @@ def resolve_config(model_or_id):
     q35 = _q35()
     if q35.config.is_supported_qwen3_5_model_id(model_or_id):
         return q35.config.make_config(model_or_id).text_config
-    if letitar_registry.is_supported_letitar_model_id(model_or_id):
-        return letitar_registry.build_config(model_or_id)
-    hf_cfg = load_hf_config_from_source(model_or_id)
-    if is_letitar_config(hf_cfg):
-        return letitar_registry.build_config(model_or_id)
+    family = stream_registry.family_of_preset(model_or_id)
+    if family is None:
+        hf_cfg = load_hf_config_from_source(model_or_id)
+        family = stream_registry.family_for(hf_cfg)
+    if family is not None:
+        return family.make_config(model_or_id)
     mt = hf_cfg.get("model_type")
     if mt in {"qwen3", "qwen3_moe"}:
         return qwen3_registry.make_config_from_hf(hf_cfg)
@@ -69,7 +70,7 @@ def resolve_config(model_or_id):
     raise ValueError(
         f"Unsupported text model/config source '{model_or_id}'. Supported Qwen3 ids: "
         f"{sorted(set(list_qwen3_dense_model_ids() + list_qwen3_moe_model_ids()))}; supported Qwen3.5 ids: "
-        f"{q35.config.list_supported_qwen3_5_model_ids()}; Letitar ids: {letitar_registry.list_letitar_model_ids()}.")
+        f"{q35.config.list_supported_qwen3_5_model_ids()}; serving decoder ids: {stream_registry.list_model_ids()}.")
 
 
 def align_config_to_mesh(cfg, mesh: Mesh):
@@ -92,8 +93,8 @@ def shard_batch_dict(batch: dict, cfg, mesh: Mesh | None = None, device=None) ->
 def model_class_for(cfg):
     if isinstance(cfg, ModelConfig):
         return Qwen3
-    if isinstance(cfg, letitar_registry.LetitarConfig):
-        return Letitar
+    if isinstance(cfg, StreamDecoderConfig):
+        return stream_registry.family_of(cfg).model_cls
     if _is_q35_text(cfg):
         return _q35().model.Qwen3_5ForCausalLM
     raise ValueError(f"Unsupported text config type: {type(cfg)}")
@@ -101,7 +102,7 @@ def model_class_for(cfg):
 
 def is_inference_only(cfg) -> bool:
     """The family's kernels have no backward pass."""
-    return isinstance(cfg, letitar_registry.LetitarConfig)
+    return isinstance(cfg, StreamDecoderConfig)
 
 
 def init_model(model_or_id, rng: int = 0, *, tp_size: int | None = None, fsdp_size: int | None = None,
@@ -130,10 +131,8 @@ def load_model(source, *, device=None, dtype=torch.bfloat16):
     """Model and config from a folder with config.json and safetensors; the class follows config.json."""
     cfg = resolve_config(str(source))
     device = device or ("cuda" if torch.cuda.is_available() else "cpu")
-    if isinstance(cfg, letitar_registry.LetitarConfig):
-        from ..models.letitar.loader import create_letitar_from_safetensors
-
-        return create_letitar_from_safetensors(source, device=device, dtype=dtype), cfg
+    if isinstance(cfg, StreamDecoderConfig):
+        return stream_registry.family_of(cfg).load_model(source, device=device, dtype=dtype), cfg
     if isinstance(cfg, ModelConfig):
         from ..models.qwen3.loader import create_qwen3_from_safetensors
 
@@ -144,8 +143,8 @@ def load_model(source, *, device=None, dtype=torch.bfloat16):
 def decode(model, cache: Cache, token_ids_BT, pad_id: int, cfg, select=None):
     """One prefill / decode call: logits [B,V] at the last non-pad column, the cache, aux.  With a paged
     cache, ``select`` (bool [B,T]) asks for the logits of the marked tokens instead, in order."""
-    if not isinstance(model, (Qwen3, Letitar)):
-        raise NotImplementedError("decode is only implemented for Qwen3 and Letitar text models.")
+    if not isinstance(model, (Qwen3, StreamDecoder)):
+        raise NotImplementedError("decode is only implemented for Qwen3 and the serving decoders (Letitar, Difedra).")
     segment_ids = (token_ids_BT != pad_id).to(torch.int32)
     if isinstance(cache, PagedSequences):
         hidden = model.decode_paged(token_ids_BT, segment_ids, cache, select)
@@ -172,16 +171,16 @@ def make_cache(cfg, batch_size: int, token_len: int, generate_steps: int, dtype=
                paged: bool | None = None, page_size: int = 64, tp_size: int = 1, num_pages: int | None = None):
     """KV cache for ``decode``.  On CUDA with bf16 (head_dim 128) the paged cache + decode kernels
     are used by default; otherwise the contiguous power-of-two cache of the reference.  With
-    ``tp_size`` > 1 the (contiguous) cache holds this tensor-parallel rank's kv heads.  Letitar models
+    ``tp_size`` > 1 the (contiguous) cache holds this tensor-parallel rank's kv heads.  Serving decoders
     use a ``HybridCache`` in ``dtype``; ``num_pages`` bounds the pages of a paged cache when the
     sequences together hold fewer tokens than batch_size full ones."""
-    if isinstance(cfg, letitar_registry.LetitarConfig):
+    if isinstance(cfg, StreamDecoderConfig):
         if tp_size > 1:
-            raise NotImplementedError("Letitar has no tensor-parallel layout")
-        return Letitar.make_cache_for(cfg, batch_size, token_len + generate_steps, page_size=page_size, num_pages=num_pages,
+            raise NotImplementedError("the serving decoders have no tensor-parallel layout")
+        return StreamDecoder.make_cache_for(cfg, batch_size, token_len + generate_steps, page_size=page_size, num_pages=num_pages,
                                       dtype=dtype, device=device)
     if not isinstance(cfg, ModelConfig):
-        raise NotImplementedError("Cache is only available for Qwen3 and Letitar text models.")
+        raise NotImplementedError("Cache is only available for Qwen3 text models and the serving decoders.")
     if tp_size > 1:
         import dataclasses
 

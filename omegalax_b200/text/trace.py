@@ -57,7 +57,7 @@ class TraceRunner:
             for b, w in enumerate(wants):
                 select[b, w] = True
             w0 = next(self.model.parameters())
-            dev_ids = ids if isinstance(self.model, api.Letitar) else ids.to(w0.device)
+            dev_ids = ids if isinstance(self.model, api.StreamDecoder) else ids.to(w0.device)
             logits, self.cache, _ = api.decode(self.model, self.cache, dev_ids, api.NO_TOKEN, self.cfg, select=select)
             place = {bt: i for i, bt in enumerate(map(tuple, select.nonzero().tolist()))}
             order = [place[(self.row[e["id"]], t)] for e in entries for t in e["want"]]
@@ -83,10 +83,11 @@ def main(argv=None) -> int:
 
     torch.backends.cuda.matmul.allow_tf32 = False
     cfg = api.resolve_config(a.model)
-    if a.dtype == "float32" and not isinstance(cfg, api.letitar_registry.LetitarConfig):
+    serving = isinstance(cfg, api.StreamDecoderConfig)
+    if a.dtype == "float32" and not serving:
         print("this model's paged decode path runs in bfloat16 only", file=sys.stderr)
         return 3
-    lib.load("serving" if isinstance(cfg, api.letitar_registry.LetitarConfig) else None)
+    lib.load(api.stream_registry.family_of(cfg).kernels if serving else None)
     torch.cuda.set_device(0)
     model, cfg = api.load_model(a.model, device=torch.device("cuda", 0), dtype=getattr(torch, a.dtype))
     runner = TraceRunner(model, cfg, a.max_tokens)

@@ -6,7 +6,8 @@ import pytest
 import torch
 
 from omegalax_b200 import export, registry
-from omegalax_b200.models.letitar.config import config_to_hf, make_config, make_config_from_hf
+from omegalax_b200.models.letitar.config import config_to_hf, make_config_from_hf
+from omegalax_b200.models.letitar.registry import FAMILY
 from omegalax_b200.models.mixers import GatedLinearAttentionConfig, LatentAttentionConfig, TokenBatch
 from omegalax_b200.models.paged_sequences import HybridCache, LatentPages, RecurrentState, SharedWith
 from omegalax_b200.models.rope_scaling import RotaryConfig, RotaryTable, YarnScaling
@@ -63,7 +64,7 @@ def test_registry_and_presets():
     assert api.model_class_for(cfg).__name__ == "Letitar"
     kinds = {type(layer.mixer) for layer in cfg.layers}
     assert kinds == {GatedLinearAttentionConfig, LatentAttentionConfig}
-    big = make_config("letitar-8layer-4096")
+    big = FAMILY.make_config("letitar-8layer-4096")
     assert big.width == 4096 and big.layers[-1].mixer.kv_from == 4
     with pytest.raises(NotImplementedError):
         api.make_cache(cfg, 1, 8, 8, tp_size=2)
@@ -146,7 +147,7 @@ def test_trace_runner_protocol(monkeypatch):
     """Rows, wanted places and freed requests, with the model's step replaced by a recorder."""
     from omegalax_b200.text import trace
 
-    cfg = make_config("letitar-smoke")
+    cfg = FAMILY.make_config("letitar-smoke")
     calls = []
 
     class Fake(torch.nn.Module):
