@@ -166,6 +166,11 @@ SERVE_PROMPTS = [(1, 8192), (8, 1024), (1, 512)]            # (sequences, tokens
 SERVE_DECODE = [(1, 4096), (32, 4096), (128, 1024)]         # (sequences, tokens already cached)
 
 
+# a serving decoder, and the model it resembles most, cut to as many layers
+SERVE_MODELS = {"letitar": ("letitar-8layer-4096", "Qwen/Qwen3-8B"),
+                "difedra": ("difedra-8layer-2048", "Qwen/Qwen3-30B-A3B-Instruct-2507")}
+
+
 def serve_bench(args) -> int:
     """Throughput of ``text.api.decode`` with a paged cache, random weights and ids: whole prompts from an
     empty cache, and single-token steps.  Each call is timed with CUDA events around it, so the copy of
@@ -181,13 +186,14 @@ def serve_bench(args) -> int:
     torch.cuda.set_device(0)
     dev = torch.device("cuda", 0)
     steps, warmup = max(args.steps, 1), max(args.warmup, 3)
-    for name in ("letitar-8layer-4096", "Qwen/Qwen3-8B"):
+    for name in SERVE_MODELS[args.serve]:
         cfg = text_api.resolve_config(name)
         if name.startswith("Qwen"):
             cfg = dataclasses.replace(cfg, num_layers=8)
         model, cfg = text_api.init_model(cfg, 0, tp_size=1, fsdp_size=1, dp_size=1, device=dev, dtype=torch.bfloat16)
-        weight_bytes = sum(p.numel() for n, p in model.named_parameters() if "embed" not in n) * 2
-        host_ids = name.startswith("letitar")
+        tied = not hasattr(model, "lm_head")      # the embedding is then also the head's matrix
+        weight_bytes = sum(p.numel() for n, p in model.named_parameters() if tied or "embed" not in n) * 2
+        host_ids = isinstance(cfg, text_api.StreamDecoderConfig)
         gen = torch.Generator().manual_seed(0)
 
         def ids(B, T):
@@ -285,9 +291,10 @@ def main() -> int:
                     help="a2a: token exchange by library all_to_all instead of the peer-memory kernels")
     ap.add_argument("--kernel-table", default=None,
                     help="after the timed regions, trace one more step and write its per-kernel device times here")
-    ap.add_argument("--serve", action="store_true",
+    ap.add_argument("--serve", nargs="?", const="letitar", choices=sorted(SERVE_MODELS),
                     help="instead of the training benchmark: prompt and decode throughput of an 8-layer Letitar and of "
-                         "an 8-layer Qwen3-8B (same width, heads and feed-forward arithmetic) on one GPU, one JSON line each")
+                         "an 8-layer Qwen3-8B, or of an 8-layer Difedra and of an 8-layer Qwen3-30B-A3B (same width, heads "
+                         "and active feed-forward arithmetic) on one GPU, one JSON line each")
     args = ap.parse_args()
     if args.serve:
         return serve_bench(args)

@@ -32,7 +32,7 @@ class DifedraConfig(StreamDecoderConfig):
                 raise ValueError(f"layer {i}: a window of {m.window} tokens")
             if m.v_from is not None and m.v_from != i:
                 src = self.layers[m.v_from].mixer if 0 <= m.v_from < i else None
-                if src is None or src.v_from != m.v_from or src.kv_heads * src.vdim != m.kv_heads * m.vdim:
+                if src is None or src.v_from != m.v_from or (src.kv_heads, src.vdim) != (m.kv_heads, m.vdim):
                     raise ValueError(f"layer {i}: its values cannot be mixed with those of layer {m.v_from}")
 
 

@@ -278,9 +278,88 @@ def bench_serving(a, dev, flush):
     _report("  like: decode projection of as many weights", it(lambda: K.gemm(xw, ww)), None, 2.0 * H * d1 * R)
 
 
+def bench_window(a, dev, flush):
+    """Windowed attention and routed experts of the serving decoders, each next to the kernel of the Qwen3
+    mixture it resembles (32 heads of 128 over --kv-heads, 8 of 128 experts of 768)."""
+    from . import moe
+    from . import serving as S
+
+    it = lambda fn: timeit(fn, a.iters, a.warmup, flush)  # noqa: E731
+    rn = lambda *s: torch.randn(*s, device=dev).to(bf16)  # noqa: E731
+    B, T, D, H, G, hd = a.batch, a.seq, a.cols, a.heads, a.kv_heads, 128
+    N, FF = B * T, 3 * D
+    x, w, xb = torch.randn(N, D, device=dev), rn(D), rn(N, D)
+    _report("rms norm rows fp32 -> bf16", it(lambda: S.rms_rows(x, w, 1e-5)), None, N * D * 6.0, rows=N, cols=D)
+    _report("  like: rmsnorm bf16", it(lambda: K.rmsnorm_fwd(xb, w, 1e-5, want_rstd=False)), None, N * D * 4.0)
+    gu = rn(N, 2 * FF)
+    _report("gated gelu", it(lambda: S.gated_act(gu, "gelu_tanh")), None, N * FF * 6.0, rows=N, cols=FF)
+    _report("gated silu", it(lambda: S.gated_act(gu, "silu")), None, N * FF * 6.0)
+    _report("  like: swiglu", it(lambda: K.swiglu_fwd(gu)), None, N * FF * 6.0)
+    del gu
+    # q, k, v preparation
+    pitch = (H + 2 * G) * hd
+    proj, first = rn(N, pitch), rn(N, G * hd)
+    pos = (torch.arange(N, device=dev) % T).to(torch.int32)
+    row = torch.arange(N, device=dev, dtype=torch.int32)
+    cos = torch.rand(T, hd // 2, device=dev)
+    nw, cache, mix = rn((H + G) * hd), rn(N, 2 * G * hd), torch.tensor(0.3, device=dev).to(bf16)
+    _report("window prepare (norms, rotation, value mixing, store)",
+            it(lambda: S.window_prepare(proj, pos, row, cos, cos, H, G, hd, hd, nw, cache, 1e-6, mix=mix, v_first=first)), None,
+            2.0 * N * hd * (2 * (H + G) + 2 * G + G + 2 * G))
+    one, c3 = rn(128), torch.randn(N, 64, device=dev)
+    _report("  like: qk-norm + rope", it(lambda: K.qknorm_rope_fwd(proj, one, one, c3, c3, H, G, hd, hd, 1e-6)), None,
+            4.0 * N * (H + G) * hd)
+    # prompt attention
+    cu = torch.arange(B + 1, device=dev, dtype=torch.int32) * T
+    q, k, v = proj[:, :H * hd], proj[:, H * hd:(H + G) * hd], proj[:, (H + G) * hd:]
+    sink = rn(H)
+    for window in (0, 4096, 1024, 128):
+        w_ = min(window or T, T)
+        pairs = B * (w_ * (w_ + 1) / 2 + (T - w_) * w_)          # (query, visible key)
+        _report(f"window attention, prompt, window {window or 'all'}",
+                it(lambda: S.attn_window(q, k, v, cu, T, H, G, hd, hd, 0.09, window, sink)), 4.0 * pairs * H * hd, None, batch=B, seq=T)
+    q3, k3, v3 = q.unflatten(1, (H, hd)), k.unflatten(1, (G, hd)), v.unflatten(1, (G, hd))
+    _report("  like: attention fwd", it(lambda: K.attn_fwd(q3, k3, v3, cu, T, 0.09, True, want_lse=False)), 2.0 * B * T * T * H * hd, None)
+    del proj, first, cache, q, k, v, q3, k3, v3, c3
+    # experts, prompts
+    E, top, F = 128, 8, 768
+    guw, dw, rw = rn(E, 2 * F, D) * 0.02, rn(E, D, F) * 0.02, rn(E, D)
+    z = torch.randn(N, E, device=dev)
+    zb = z.to(bf16)
+    _report("sigmoid router", it(lambda: S.route_sigmoid(z, top)), None, N * (E * 4.0 + top * 8))
+    _report("  like: softmax router", it(lambda: K.router_topk(zb, top, True)), None, N * (E * 6.0 + top * 8))
+    wt, idx = S.route_sigmoid(z, top)
+    fl = 6.0 * N * top * D * F
+    _report("experts, prompt (plan, gather, products, gate, sum)", it(lambda: S.experts_into(xb, wt, idx, guw, dw, "silu", x)), fl, None, rows=N)
+    i64 = idx.long()
+    with torch.no_grad():
+        _report("  like: expert mixture", it(lambda: moe.moe_mlp(xb, wt, i64, guw, dw)), fl, None)
+    # decode
+    Bd, ctx, page = a.decode_batch, a.ctx, 64
+    seen = torch.full((Bd,), ctx, dtype=torch.int32, device=dev)
+    blocks = -(-(ctx + 1) // page)
+    table = torch.randperm(Bd * blocks, device=dev).to(torch.int32).view(Bd, blocks)
+    rows_, qd = rn(Bd * blocks * page, 2 * G * hd), rn(Bd, H * hd)
+    for window in (0, 1024, 128):
+        _report(f"window decode attention, window {window or 'all'}",
+                it(lambda: S.window_decode(qd, rows_, seen, table, page, H, G, hd, hd, 0.09, window, sink)), None,
+                4.0 * Bd * min(window or ctx, ctx) * G * hd, batch=Bd, ctx=ctx)
+    kp, vp, qq = rn(Bd * blocks, page, G, hd), rn(Bd * blocks, page, G, hd), rn(Bd, H, hd)
+    _report("  like: paged decode attention", it(lambda: K.decode_attn(qq, kp, vp, table, seen, page, 0.09)), None, 4.0 * Bd * ctx * G * hd)
+    hb, xd = rn(Bd, D), torch.randn(Bd, D, device=dev)
+    wt, idx = S.route_sigmoid(torch.randn(Bd, E, device=dev), top)
+    by = 6.0 * idx.unique().numel() * D * F                      # weights of the experts that are used
+    _report("experts, decode", it(lambda: S.experts_into(hb, wt, idx, guw, dw, "silu", xd)), None, by, batch=Bd)
+    i64 = idx.long()
+    with torch.no_grad():
+        _report("  like: expert mixture", it(lambda: moe.moe_mlp(hb, wt, i64, guw, dw)), None, by)
+    _report("  (grouped products instead)", it(lambda: S.experts_into(hb, wt, idx, guw, dw, "silu", xd, few=False)), None, by)
+    _report("router product", it(lambda: S.project(hb, rw, out_dtype=torch.float32)), None, 2.0 * E * D)
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "attn", "gdn", "decode", "elementwise", "ce", "serving"])
+    ap.add_argument("what", choices=["gemm", "attn", "gdn", "decode", "elementwise", "ce", "serving", "window"])
     ap.add_argument("--m", type=int, default=16384)
     ap.add_argument("--n", type=int, default=6144)
     ap.add_argument("--k", type=int, default=4096)
@@ -303,7 +382,7 @@ def main():
     torch.cuda.set_device(dev)
     flush = torch.zeros(64 * 1024 * 1024, device=dev) if a.iters > 0 else None
     {"gemm": bench_gemm, "attn": bench_attn, "gdn": bench_gdn, "decode": bench_decode,
-     "elementwise": bench_elementwise, "ce": bench_ce, "serving": bench_serving}[a.what](a, dev, flush)
+     "elementwise": bench_elementwise, "ce": bench_ce, "serving": bench_serving, "window": bench_window}[a.what](a, dev, flush)
     torch.cuda.synchronize()
     lib.check_status()
 
