@@ -51,6 +51,13 @@ struct AttnFwdArgs {
   int* status;
 };
 
+// bits lo ... hi (inclusive, any integers) of a 32-bit word
+__device__ __forceinline__ uint32_t bits_between(int lo, int hi) {
+  const uint32_t upto = hi >= 31 ? 0xffffffffu : hi < 0 ? 0u : (2u << hi) - 1u;
+  const uint32_t from = lo <= 0 ? 0xffffffffu : lo > 31 ? 0u : 0xffffffffu << lo;
+  return upto & from;
+}
+
 template <int QB, int VB, int KST, int VST>
 struct AttnFwdSmem {
   static constexpr int kQTile = 128 * QB * 64 * 2;    // one 128-row query / key tile
@@ -106,7 +113,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     else n_w[w] = p.causal ? min(n_kv_total, (qs >> 7) + 1) : n_kv_total;
   }
   const int n = max(n_w[0], n_w[1]);
-  const int j_lo = lo_w[0];        // the first rows see furthest back
+  const int j_lo = kWindow ? lo_w[0] : 0;        // the first rows see furthest back
+  auto lo_of = [&](int w) { return kWindow ? lo_w[w] : 0; };
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < 2; ++i) {
@@ -196,7 +204,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       };
       bool ok = mbar_wait(&k_full[0], 0, abort_flag, p.status, OB_ERR_WAIT_FULL);
       for (int w = 0; w < 2 && ok; ++w) {
-        if (n_w[w] > 0 && lo_w[w] == j_lo) {
+        if (n_w[w] > 0 && lo_of(w) == j_lo) {
           ok = mbar_wait(&q_full[w], 0, abort_flag, p.status, OB_ERR_WAIT_FULL);
           if (!ok) break;
           tc_fence_after();
@@ -213,21 +221,21 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         bool k_next_ready = false;
         for (int w = 0; w < 2 && ok; ++w) {
           if (j >= n_w[w]) continue;
-          if (j >= lo_w[w]) {
-            ok = mbar_wait(&p_ready[w], (j - lo_w[w]) & 1, abort_flag, p.status, OB_ERR_WAIT_MISC);
+          if (j >= lo_of(w)) {
+            ok = mbar_wait(&p_ready[w], (j - lo_of(w)) & 1, abort_flag, p.status, OB_ERR_WAIT_MISC);
             if (!ok) break;
             tc_fence_after();
-            issue_pv(w, s, j == lo_w[w]);
+            issue_pv(w, s, j == lo_of(w));
             umma_commit(&o_full[w]);
           }
-          if (j + 1 >= lo_w[w] && j + 1 < n_w[w]) {
+          if (j + 1 >= lo_of(w) && j + 1 < n_w[w]) {
             if (!k_next_ready) {
               ok = mbar_wait(&k_full[kn], ((t + 1) / KST) & 1, abort_flag, p.status, OB_ERR_WAIT_FULL);
               if (!ok) break;
               tc_fence_after();
               k_next_ready = true;
             }
-            if (j + 1 == lo_w[w]) {      // (kWindow) this warpgroup's first tile
+            if (kWindow && j + 1 == lo_of(w)) {      // this warpgroup's first tile
               ok = mbar_wait(&q_full[w], 0, abort_flag, p.status, OB_ERR_WAIT_FULL);
               if (!ok) break;
               tc_fence_after();
@@ -256,7 +264,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     constexpr float kRescaleLog2 = 8.f;
     float m_ref = -INFINITY, m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
-    const int nj = n_w[w], lo = lo_w[w];
+    const int nj = n_w[w], lo = lo_of(w);
     const int kfirst = kWindow && p.window > 0 ? max(0, qpos - p.window + 1) : 0;    // first visible key
     for (int j = lo; j < nj && ok; ++j) {
       ok = mbar_wait(&s_full[w], (j - lo) & 1, abort_flag, p.status, OB_ERR_WAIT_TMEM_FULL);
@@ -273,10 +281,14 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         uint32_t v[32];
         tmem_ld32(s_addr + c * 32, v);
         tmem_ld_wait();
-        if (need_mask) {
+        if (kWindow && need_mask) {
+          const uint32_t seen = bits_between(kfirst - kbase - c * 32, klimit - kbase - c * 32);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) mx = fmaxf(mx, (seen >> i) & 1 ? __uint_as_float(v[i]) : -INFINITY);
+        } else if (need_mask) {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (kbase + c * 32 + i <= klimit && (!kWindow || kbase + c * 32 + i >= kfirst)) mx = fmaxf(mx, __uint_as_float(v[i]));
+            if (kbase + c * 32 + i <= klimit) mx = fmaxf(mx, __uint_as_float(v[i]));
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) mx = fmaxf(mx, __uint_as_float(v[i]));
@@ -316,14 +328,20 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         tmem_ld32(s_addr + c * 32, v);
         tmem_ld_wait();
         uint32_t pk[16];
+        uint32_t seen = 0xffffffffu;
+        if (kWindow && need_mask) seen = bits_between(kfirst - kbase - c * 32, klimit - kbase - c * 32);
+        if (kWindow && seen != 0xffffffffu) {      // hidden scores become -inf, their exponentials 0
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (!((seen >> i) & 1)) v[i] = 0xff800000u;
+        }
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           float p0 = fast_exp2(__uint_as_float(v[2 * i]) * p.scale_log2 - m_safe);
           float p1 = fast_exp2(__uint_as_float(v[2 * i + 1]) * p.scale_log2 - m_safe);
-          if (need_mask) {
-            const int k0 = kbase + c * 32 + 2 * i;
-            if (k0 > klimit || (kWindow && k0 < kfirst)) p0 = 0.f;
-            if (k0 + 1 > klimit || (kWindow && k0 + 1 < kfirst)) p1 = 0.f;
+          if (!kWindow && need_mask) {
+            if (kbase + c * 32 + 2 * i > klimit) p0 = 0.f;
+            if (kbase + c * 32 + 2 * i + 1 > klimit) p1 = 0.f;
           }
           lsum += p0 + p1;
           pk[i] = pack_bf16(p0, p1);

@@ -320,6 +320,10 @@ def bench_window(a, dev, flush):
                 it(lambda: S.attn_window(q, k, v, cu, T, H, G, hd, hd, 0.09, window, sink)), 4.0 * pairs * H * hd, None, batch=B, seq=T)
     q3, k3, v3 = q.unflatten(1, (H, hd)), k.unflatten(1, (G, hd)), v.unflatten(1, (G, hd))
     _report("  like: attention fwd", it(lambda: K.attn_fwd(q3, k3, v3, cu, T, 0.09, True, want_lse=False)), 2.0 * B * T * T * H * hd, None)
+    if N % 256 == 0:        # as few tiles per query block as a window of 128 leaves
+        cu_s = torch.arange(N // 256 + 1, device=dev, dtype=torch.int32) * 256
+        _report("  like: attention fwd, sequences of 256", it(lambda: K.attn_fwd(q3, k3, v3, cu_s, 256, 0.09, True, want_lse=False)),
+                2.0 * N * 256 * H * hd, None)
     del proj, first, cache, q, k, v, q3, k3, v3, c3
     # experts, prompts
     E, top, F = 128, 8, 768
