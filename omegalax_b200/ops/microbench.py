@@ -8,6 +8,7 @@ flush between timed launches, reported against the measured peaks of the box.
     python -m omegalax_b200.ops.microbench elementwise --rows 32768 --cols 4096
     python -m omegalax_b200.ops.microbench ce --rows 8192 --vocab 151936
     python -m omegalax_b200.ops.microbench serving --batch 2 --seq 8192 --ctx 4096
+    python -m omegalax_b200.ops.microbench window --batch 2 --seq 8192 --cols 2048 --kv-heads 4
 
 ``--iters 0 --warmup N`` only launches the kernels N times (for a profiler capture of a small
 case); ``--baseline`` also times the library counterpart (cuBLAS / SDPA) for comparison.

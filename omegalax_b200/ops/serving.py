@@ -326,10 +326,11 @@ def window_decode_fits(dtype, dim: int, vdim: int) -> bool:
 
 
 def window_decode_splits(B: int, H: int, G: int, keys: int) -> int:
-    """Key splits per sequence and key/value head: about two CTAs per SM, at least one 64-key tile each."""
+    """Key splits per sequence and key/value head: about two CTAs per SM, at least two 64-key tiles each
+    (a tile costs a CTA 2 us, merging the splits 4)."""
     R = H // G
     blocks = B * G * -(-R // (16 if R <= 16 else 32))
-    return max(1, min(296 // blocks, keys // 64, 64))
+    return max(1, min(296 // blocks, keys // 128, 64))
 
 
 def window_decode(q, cache, seen, block_table, page_size: int, H: int, G: int, dim: int, vdim: int, scale: float, window: int,
